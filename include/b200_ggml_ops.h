@@ -25,7 +25,7 @@ enum b200_binary_op { B200_BIN_ADD = 0, B200_BIN_SUB = 1, B200_BIN_MUL = 2, B200
 enum b200_unary_op {
     B200_UN_SILU = 0, B200_UN_GELU = 1, B200_UN_GELU_QUICK = 2, B200_UN_RELU = 3, B200_UN_TANH = 4, B200_UN_SIGMOID = 5,
     B200_UN_SQR = 6, B200_UN_SCALE = 7 /* p0 = factor */, B200_UN_CLAMP = 8 /* p0 = min, p1 = max */,
-    B200_UN_SOFTCAP = 9 /* p0 * tanh(x / p0) */,
+    B200_UN_SOFTCAP = 9 /* p0 * tanh(x / p0) */, B200_UN_RELU_SQR = 10 /* max(x, 0)^2 */,
 };
 
 /* RMS_NORM (+ optional fused MUL by a per-column weight): y = x / sqrt(mean(x^2) + eps) [* w]
@@ -74,7 +74,7 @@ B200_API int b200_op_rope_kv_store(const b200_tensor *q, const b200_tensor *q_ds
                                    const b200_tensor *v, const int32_t *pos, const float *freq_factors, const b200_rope_params *rp,
                                    int kv_type, void *k_cache, void *v_cache, void *const *k_slot, void *const *v_slot, b200_stream_t stream);
 
-/* GET_ROWS: dst[i] = dequantise(src row ids[i]); src f32 / f16 / q4_0 / q8_0 / q4_K / q5_K / q6_K (K-quant token embeddings
+/* GET_ROWS: dst[i] = dequantise(src row ids[i]); src i32 (dst i32, a table of integers) / f32 / f16 / q4_0 / q8_0 / q4_K / q5_K / q6_K (K-quant token embeddings
  * stay on the device -- the reference falls back to the CPU for them, ggml-cuda.cu:3033-3047).
  * replaces k_get_rows / k_get_rows_float, ggml-cuda/getrows.cu:5-120 */
 B200_API int b200_op_get_rows(const b200_tensor *src, const b200_tensor *ids, const b200_tensor *dst, b200_stream_t stream);
@@ -122,12 +122,13 @@ enum b200_ext_op {
     B200_EXT_MLSTM_SCAN = 8,   /* src: q, k, v, ig, fg, i_bias, f_bias, seq_info, state; op_params: [2] heads, [3] dim, [4] vdim, [5] gate_cap */
     B200_EXT_QKV_STORE = 9,    /* src: q, k, v, vecs (the present ones of q.b, k.b, v.b, q.norm, k.norm packed in one tensor, or NULL), pos, freqs,
                                   cells, k cache, v cache; q in place; op_params: [2] dim, [3] vdim, [4] n_dims, [5] eps, [6] biases present, [7] norms present
-                                  (1: over the whole row, 2: per head with one weight vector of dim values), [8] pairs are (i, i + n_dims / 2), [9] every head of v is divided
+                                  (1: over the whole row, 2: per head with one weight vector of dim values, 3: per head without a weight), [8] pairs are (i, i + n_dims / 2), [9] every head of v is divided
                                   by its root mean square, [10] q temperature coefficient, [11] its period in positions; freqs may be NULL without rotation */
     B200_EXT_SINK_ATTN = 10,   /* src: q, k cache, v cache, sink, tok_seq, tok_pos, cell_seq, cell_pos, [head gate [heads, T]]; op_params: [2] dim, [3] scale,
-                                  [4] window, [5] keep_first, [6] bf16 products, [7] vdim, [8] chunk, [9] enum b200_attn_weights; src[9]: score bias by distance
-                                  [n_dist, heads] (optional) */
-    B200_EXT_LINEAR_ATTN_SCAN = 11, /* src: q, k, v, decay, seq_info, state; op_params: [2] heads, [3] dim, [4] vdim, [5] silu on q / k / v */
+                                  [4] window, [5] keep_first, [6] bf16 products, [7] vdim, [8] chunk, [9] enum b200_attn_weights, [10] linear distance bias, [11] factor on
+                                  the result (0 reads as 1); src[8] of [heads * vdim, T]: a gate per value; src[9]: score bias by distance [n_dist, heads] (optional) */
+    B200_EXT_LINEAR_ATTN_SCAN = 11, /* src: q, k, v, decay, seq_info, state, [pos, freqs]; op_params: [2] heads, [3] dim, [4] vdim, [5] silu on q / k / v, [6] factor on k
+                                  (0 reads as 1), [7] n_dims of the rotation (0: none) */
     B200_EXT_MOE_ROUTE = 12,   /* src: logits, correction; dst [2 n_used, T]: per token n_used weights (f32), then n_used expert ids (i32);
                                   op_params: [2] n_group, [3] n_group_used, [4] scale, [5] n_used, [6] enum b200_router_score, [7] weights are the
                                   scores as they are (no division by their sum) */
@@ -145,6 +146,10 @@ enum b200_ext_op {
                                   unit vectors, [7] the eps of that, [8] q scale */
     B200_EXT_MINGRU_SCAN = 20, /* src: z, x, g (optional), z bias, x bias (optional), seq_info, state [width, slots] */
     B200_EXT_NORM_PAIR = 21,   /* src: x1, w1, b1 (optional), x2, w2: dst = N(x1 + b1) * w1 + N(x2) * w2, N the RMS norm; op_params: [3] eps */
+    B200_EXT_NORM_CHAIN = 22,  /* src: y [n, n_y, T], y weights [n_y, T] (optional), shared [n, T] (optional), res [n, T] (optional), w1, b1, w2, b2 (optional each);
+                                  dst [n, T, 1 or 2]: x, then h (b200_op_norm_chain); op_params: [2] kind1, [3] eps, [4] kind2, [5] y scale (0 reads as 1) */
+    B200_EXT_TOKEN_SHIFT = 23, /* src: h [n, T], mu [n, n_mix], seq_info, prev [n, slots]; dst [n, T, n_mix] (b200_op_token_shift) */
+    B200_EXT_TIME_MIX_SCAN = 24, /* src: r, k, v, z, w0, u, seq_info, state; op_params: [2] heads, [3] dim (b200_op_time_mix_scan) */
 };
 /* how attention turns scores into weights: SOFTMAX over the visible keys (with the sink in the denominator), or SIGMOID of every score by
  * itself with no normalisation over the keys (a sink has no meaning then) */
@@ -172,6 +177,24 @@ B200_API int b200_op_norm_affine(const b200_tensor *x, const float *w, int64_t w
  * over ne0; b1 optional; x1, x2, dst f32 rows of one shape with any row strides; ne0 <= 16384. */
 B200_API int b200_op_norm_pair(const b200_tensor *x1, const float *w1, const float *b1, const b200_tensor *x2, const float *w2, const b200_tensor *dst, float eps,
                                b200_stream_t stream);
+
+/* A sublayer's result behind its norm, the residual stream, and the next sublayer's input norm in one launch, a token per CTA:
+ *   s = y_scale * sum_k yw[t][k] * y[t][k] + shared[t]      (yw NULL: weights of one; shared optional; n_y = 1 for a plain result)
+ *   x[t] = res[t] + N1(s) * w1 + b1,   h[t] = N2(x[t]) * w2 + b2   (h NULL: not wanted)
+ * N1, N2: enum b200_norm_kind with the same eps; w1, b1, w2, b2, res optional.  Strides in floats; n <= 16384. */
+typedef struct {
+    const float *y; int64_t y_s_slot, y_s_tok;
+    const float *yw; int64_t yw_s_tok;
+    const float *shared; int64_t shared_stride;
+    const float *res; int64_t res_stride;
+    const float *w1, *b1, *w2, *b2;
+    float *x; int64_t x_stride;
+    float *h; int64_t h_stride;
+    int64_t n, n_tok;
+    int32_t n_y, kind1, kind2;
+    float y_scale, eps;
+} b200_norm_chain_args;
+B200_API int b200_op_norm_chain(const b200_norm_chain_args *a, b200_stream_t stream);
 
 /* PolyNorm: dst = c0 N(x) + c1 N(x^2) + c2 N(x^3) + c3 with N(z) = z / sqrt(mean(z^2) + eps) over ne0, powers element by
  * element; coef: 4 floats on the device. */
@@ -267,6 +290,7 @@ typedef struct {
     int32_t v_unit_rms;                    /* 1: every head of v is divided by sqrt(mean(v^2) + eps) before it is stored (behind the bias) */
     float   q_temp_coef;                   /* != 0: q is multiplied by 1 + coef * ln(floor((pos + 1) / q_temp_every) + 1) */
     int32_t q_temp_every;
+    int32_t qk_unit_rms;                   /* 1: every head of q and k is divided by sqrt(mean(x^2) + eps), no weight */
 } b200_qkv_store_args;
 B200_API int b200_op_qkv_store(const b200_qkv_store_args *a, b200_stream_t stream);
 
@@ -289,6 +313,9 @@ typedef struct {
     const float *gate; int64_t gate_stride;
     int32_t weights;                       /* enum b200_attn_weights */
     const float *dist_bias; int32_t n_dist; /* [n_head][n_dist] added to the scaled score of a key min(tok_pos - cell_pos, n_dist - 1) positions back (NULL: none) */
+    int32_t dist_linear;                   /* 1: dist_bias[h][0] is a bias per position instead: dist_bias[h][0] * (tok_pos - cell_pos) joins the score */
+    int32_t gate_per_value;                /* 1: gate has n_head * vdim values per token, one for every value of the result */
+    float   out_scale;                     /* the result is multiplied by this (0 reads as 1) */
 } b200_sink_attn_args;
 B200_API int b200_op_sink_attn(const b200_sink_attn_args *a, b200_stream_t stream);
 /* The same with a workspace of b200_sink_attn_workspace_bytes(a) bytes (16-byte aligned; 0: none needed): with few tokens and
@@ -297,7 +324,7 @@ B200_API size_t b200_sink_attn_workspace_bytes(const b200_sink_attn_args *a);
 B200_API int b200_op_sink_attn_ws(const b200_sink_attn_args *a, void *workspace, size_t workspace_bytes, b200_stream_t stream);
 
 /* Linear attention with a decayed state per (slot, head), f32: S' = decay[h] S + k v^T, o = S'^T q, over the tokens of n_seq
- * sequences; act != 0 applies silu to q, k and v first.  seq_info as for b200_op_mlstm_scan.  State [head][vdim][dim] per slot.
+ * sequences; act != 0 applies silu to q, k and v first; optional rotation of q and k and a factor on k.  seq_info as for b200_op_mlstm_scan.  State [head][vdim][dim] per slot.
  * q, k: [n_tokens][heads * dim], v and dst: [n_tokens][heads * vdim]; strides in floats. */
 typedef struct {
     const float *q, *k, *v; int64_t q_stride, k_stride, v_stride;
@@ -306,6 +333,9 @@ typedef struct {
     float *state; int64_t slot_stride;
     float *dst; int64_t dst_stride;
     int32_t heads, dim, vdim, act;
+    float   k_scale;                       /* k is multiplied by this (0 reads as 1) */
+    const int32_t *pos; const float *freqs; /* n_dims > 0: entry i of every head of q and k turns with entry i + n_dims / 2 by pos[t] * freqs[i], */
+    int32_t n_dims;                        /* i < n_dims / 2, behind the activation; entries from n_dims on stay (every CTA of a head turns its own copy: for few tokens) */
 } b200_linear_attn_args;
 B200_API int b200_op_linear_attn_scan(const b200_linear_attn_args *a, b200_stream_t stream);
 
@@ -392,6 +422,33 @@ typedef struct {
     int32_t width, n_tokens;
 } b200_mingru_args;
 B200_API int b200_op_mingru_scan(const b200_mingru_args *a, b200_stream_t stream);
+
+/* Token shift: with h' the previous token's row of the same sequence (zeros in front of a fresh one), mix m of token t is
+ *   dst[m][t] = h[t] + (h'[t] - h[t]) * mu[m].
+ * The last row of a sequence waits in its slot of `prev` for the next tokens.  mu [n_mix][width]; strides in floats. */
+typedef struct {
+    const float *h; int64_t h_stride;
+    const float *mu;
+    const int32_t *seq_info; int32_t n_seq;
+    float *prev; int64_t slot_stride;
+    float *dst; int64_t dst_s_mix, dst_s_tok;
+    int32_t width, n_mix, n_tokens;
+} b200_token_shift_args;
+B200_API int b200_op_token_shift(const b200_token_shift_args *a, b200_stream_t stream);
+
+/* Linear attention whose state forgets by a decay per token and key channel, with a bonus for the current token (time mixing), f32:
+ *   w = exp(-exp(z[t] + w0));  o = (S + diag(u) k v^T)^T r;  S <- diag(w) S + k v^T.
+ * r, k, v, z [n_tokens][heads * dim]; w0, u [heads * dim]; state [head][value column][key channel] per slot; seq_info as for
+ * b200_op_mlstm_scan; strides in floats; dim <= 256. */
+typedef struct {
+    const float *r, *k, *v, *z; int64_t r_stride, k_stride, v_stride, z_stride;
+    const float *w0, *u;
+    const int32_t *seq_info; int32_t n_seq;
+    float *state; int64_t slot_stride;
+    float *dst; int64_t dst_stride;
+    int32_t heads, dim;
+} b200_time_mix_args;
+B200_API int b200_op_time_mix_scan(const b200_time_mix_args *a, b200_stream_t stream);
 
 #ifdef __cplusplus
 }

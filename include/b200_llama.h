@@ -47,17 +47,21 @@ typedef struct {
     float   residual_mult;           /* architectures that scale a sublayer's result before it joins the residual stream (0 reads as 1) */
 } b200_llama_params;
 
-enum b200_arch { B200_ARCH_LLAMA = 0, B200_ARCH_GENESUN = 1, B200_ARCH_GALIRAX = 2, B200_ARCH_ZEVOPEL = 3, B200_ARCH_MEDODRA = 4 };
+enum b200_arch { B200_ARCH_LLAMA = 0, B200_ARCH_GENESUN = 1, B200_ARCH_GALIRAX = 2, B200_ARCH_ZEVOPEL = 3, B200_ARCH_MEDODRA = 4, B200_ARCH_MAFUZEN = 5 };
 enum b200_mixer {
     B200_MIXER_LATENT_ATTENTION = 1, B200_MIXER_MLSTM = 2,
     B200_MIXER_ATTENTION = 3, /* softmax attention of heads over kv_heads cached keys / values, per-head sink, optional window */
     B200_MIXER_LIGHTNING = 4, /* linear attention: a decayed outer-product state per head */
     B200_MIXER_DELTA = 5,     /* gated delta rule: the state forgets by a per-token decay and is corrected towards v along k */
     B200_MIXER_SIGMOID_ATTENTION_GRU = 6, /* two mixers side by side: attention with sigmoid weights and a distance bias, and a minGRU */
+    B200_MIXER_RETENTION = 7, /* linear attention with a fixed decay per head, rotated queries and keys, a norm per head and a gate behind it */
+    B200_MIXER_WINDOW_ATTENTION_TIME_MIX = 8, /* two mixers side by side: windowed attention whose values are its keys, and time mixing */
 };
 enum b200_mlp {
     B200_MLP_NONE = 0, B200_MLP_DENSE_POLYNORM = 1, B200_MLP_MOE_GATED = 2 /* routed gated experts */,
     B200_MLP_DENSE_GATED = 3, /* down(act(gate x) * up x), act by glu_kind */
+    B200_MLP_MOE_TABLE = 4,   /* experts down(max(up x, 0)^2) that a table names by token id ("mlp.table" [vocab, n_expert_used], i32), each with the
+                                 weight 1 / n_expert_used; shared_ff > 0: a shared expert of the same form runs for every token */
 };
 enum b200_rope_scaling { B200_ROPE_SCALING_NONE = 0, B200_ROPE_SCALING_YARN = 1, B200_ROPE_SCALING_BANDS = 2 /* per wavelength band */ };
 
@@ -114,6 +118,12 @@ typedef struct {
     int32_t shared_ff;               /* > 0: a shared expert of this hidden size runs for every token ("mlp.shared.*"), times sigmoid(W_sg x) */
     int32_t loop_input;              /* 1: every time this layer is about to run, the stream x is first replaced by W_in [x ; x0] ("loop.in" [width, 2 width]),
                                         x0 being the stream as the embedding left it: the first layer of a looped stretch */
+    /* attention, further switches (kv_from serves B200_MIXER_ATTENTION too: the layer has queries only and reads that layer's cache) */
+    float   dist_slope_exp;          /* > 0: slope_h * distance is taken off the score, slope_h = 2^(-dist_slope_exp (h + 1) / heads) */
+    /* B200_MIXER_WINDOW_ATTENTION_TIME_MIX: heads .. keep_first describe the attention; time mixing has heads of its own */
+    int32_t mix_heads, mix_dim;
+    float   left_scale, right_scale; /* factors on the two results before they are added */
+    int32_t token_side;              /* > 0: a second embedding of this size per layer joins behind the feed-forward ("side.*") */
 } b200_layer_params;
 
 

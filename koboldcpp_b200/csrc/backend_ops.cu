@@ -76,10 +76,11 @@ static bool ext_op_supported(const ggml_tensor *op) {
         case B200_EXT_SINK_ATTN:
             return f32_rows(s[0]) && f32_rows(s[1]) && f32_rows(s[2]) && (!s[3] || f32_vec(s[3])) && i32_vec(s[4]) && i32_vec(s[5]) && i32_vec(s[6]) && i32_vec(s[7]) &&
                    f32_rows(op) && op->op_params[2] > 0 && op->op_params[2] <= 256 && op->op_params[7] > 0 && op->op_params[7] <= 256 && s[0]->ne[0] % op->op_params[2] == 0 &&
-                   (!s[8] || (f32_rows(s[8]) && s[8]->ne[0] == s[0]->ne[0] / op->op_params[2] && s[8]->ne[1] == s[0]->ne[1])) &&
+                   (!s[8] || (f32_rows(s[8]) && (s[8]->ne[0] == s[0]->ne[0] / op->op_params[2] || s[8]->ne[0] == s[0]->ne[0] / op->op_params[2] * op->op_params[7]) && s[8]->ne[1] == s[0]->ne[1])) &&
                    (!s[9] || (f32_vec(s[9]) && s[9]->ne[1] == s[0]->ne[0] / op->op_params[2] && s[9]->ne[0] > 0));
         case B200_EXT_LINEAR_ATTN_SCAN:
-            return f32_rows(s[0]) && f32_rows(s[1]) && f32_rows(s[2]) && f32_vec(s[3]) && i32_vec(s[4]) && f32_rows(s[5]) && f32_rows(op) && op->op_params[3] <= 256;
+            return f32_rows(s[0]) && f32_rows(s[1]) && f32_rows(s[2]) && f32_vec(s[3]) && i32_vec(s[4]) && f32_rows(s[5]) && f32_rows(op) && op->op_params[3] <= 256 &&
+                   (op->op_params[7] == 0 || (i32_vec(s[6]) && f32_vec(s[7])));
         case B200_EXT_MOE_ROUTE:
             return f32_rows(s[0]) && (!s[1] || f32_vec(s[1])) && f32_rows(op) && s[0]->ne[0] <= 256 && op->op_params[5] > 0 && op->op_params[5] <= 32 && op->ne[0] == 2 * op->op_params[5] &&
                    op->ne[1] == s[0]->ne[1];
@@ -112,6 +113,18 @@ static bool ext_op_supported(const ggml_tensor *op) {
         case B200_EXT_MINGRU_SCAN:
             return f32_rows(s[0]) && f32_rows(s[1]) && (!s[2] || f32_rows(s[2])) && (!s[3] || f32_vec(s[3])) && (!s[4] || f32_vec(s[4])) && i32_vec(s[5]) && f32_rows(s[6]) &&
                    f32_rows(op) && s[6]->ne[0] >= op->ne[0];
+        case B200_EXT_NORM_CHAIN:
+            if (!f32_rows(s[0]) || !f32_rows(op) || op->ne[0] != s[0]->ne[0] || op->ne[1] != s[0]->ne[2] || op->ne[0] > 16384 || op->ne[2] < 1 || op->ne[2] > 2) return false;
+            for (int i = 1; i < 4; i++) if (s[i] && !f32_rows(s[i])) return false;
+            for (int i = 4; i < 8; i++) if (s[i] && !(f32_vec(s[i]) && s[i]->ne[0] == op->ne[0])) return false;
+            return true;
+        case B200_EXT_TOKEN_SHIFT:
+            return f32_rows(s[0]) && f32_vec(s[1]) && i32_vec(s[2]) && f32_rows(s[3]) && f32_rows(op) && s[0]->ne[0] == op->ne[0] && s[0]->ne[1] == op->ne[1] &&
+                   s[1]->ne[0] == op->ne[0] && s[1]->ne[1] == op->ne[2] && s[3]->ne[0] >= op->ne[0];
+        case B200_EXT_TIME_MIX_SCAN:
+            for (int i = 0; i < 4; i++) if (!f32_rows(s[i])) return false;
+            return f32_vec(s[4]) && f32_vec(s[5]) && i32_vec(s[6]) && f32_rows(s[7]) && f32_rows(op) && op->op_params[3] > 0 && op->op_params[3] <= 256 &&
+                   nelements(s[4]) == (int64_t)op->op_params[2] * op->op_params[3] && nelements(s[5]) == nelements(s[4]);
         default:
             return false;
     }
@@ -132,6 +145,8 @@ static void fill_sink_attn_args(const ggml_tensor *n, b200_sink_attn_args &a) {
     if (s[8]) { a.gate = (const float *)s[8]->data; a.gate_stride = (int64_t)(s[8]->nb[1] / 4); }
     a.weights = n->op_params[9];
     if (s[9]) { a.dist_bias = (const float *)s[9]->data; a.n_dist = (int32_t)s[9]->ne[0]; }
+    a.dist_linear = n->op_params[10]; a.out_scale = ext_f(n, 11);
+    a.gate_per_value = s[8] && s[8]->ne[0] != a.n_head;
 }
 
 // the batched tensor-core form of an expert product over bf16 weights (the grouped GEMM of the quantised types)
@@ -224,8 +239,8 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
             const float *vec = s[3] ? (const float *)s[3]->data : nullptr;
             const int64_t nq = (int64_t)a.n_head * a.dim, nk = (int64_t)a.n_head_kv * a.dim, nv = (int64_t)a.n_head_kv * a.vdim;
             if (vec && n->op_params[6]) { a.q_bias = vec; a.k_bias = vec + nq; a.v_bias = vec + nq + nk; vec += nq + nk + nv; }
-            a.norm_per_head = n->op_params[7] == 2; a.rope_halves = n->op_params[8] != 0;
-            if (vec && n->op_params[7]) { a.q_norm = vec; a.k_norm = vec + (a.norm_per_head ? a.dim : nq); }
+            a.norm_per_head = n->op_params[7] == 2; a.qk_unit_rms = n->op_params[7] == 3; a.rope_halves = n->op_params[8] != 0;
+            if (vec && n->op_params[7] && !a.qk_unit_rms) { a.q_norm = vec; a.k_norm = vec + (a.norm_per_head ? a.dim : nq); }
             a.pos = (const int32_t *)s[4]->data; a.freqs = s[5] ? (const float *)s[5]->data : nullptr; a.cells = (const int32_t *)s[6]->data;
             a.k_cache = (float *)s[7]->data; a.k_cache_stride = (int64_t)(s[7]->nb[1] / 4);
             a.v_cache = (float *)s[8]->data; a.v_cache_stride = (int64_t)(s[8]->nb[1] / 4);
@@ -253,6 +268,8 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
             a.state = (float *)s[5]->data; a.slot_stride = (int64_t)(s[5]->nb[1] / 4);
             a.dst = (float *)n->data; a.dst_stride = (int64_t)(n->nb[1] / 4);
             a.heads = n->op_params[2]; a.dim = n->op_params[3]; a.vdim = n->op_params[4]; a.act = n->op_params[5];
+            a.k_scale = ext_f(n, 6); a.n_dims = n->op_params[7];
+            if (a.n_dims > 0) { a.pos = (const int32_t *)s[6]->data; a.freqs = (const float *)s[7]->data; }
             B200_CHECK_RC(b200_op_linear_attn_scan(&a, x.stream));
             break;
         }
@@ -361,6 +378,47 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
             B200_CHECK_RC(b200_op_mingru_scan(&a, x.stream));
             break;
         }
+        case B200_EXT_NORM_CHAIN: {
+            b200_norm_chain_args a;
+            memset(&a, 0, sizeof(a));
+            a.y = (const float *)s[0]->data; a.y_s_slot = (int64_t)(s[0]->nb[1] / 4); a.y_s_tok = (int64_t)(s[0]->nb[2] / 4); a.n_y = (int32_t)s[0]->ne[1];
+            if (s[1]) { a.yw = (const float *)s[1]->data; a.yw_s_tok = (int64_t)(s[1]->nb[1] / 4); }
+            if (s[2]) { a.shared = (const float *)s[2]->data; a.shared_stride = (int64_t)(s[2]->nb[1] / 4); }
+            if (s[3]) { a.res = (const float *)s[3]->data; a.res_stride = (int64_t)(s[3]->nb[1] / 4); }
+            const float **vecs[4] = {&a.w1, &a.b1, &a.w2, &a.b2};
+            for (int i = 0; i < 4; i++) *vecs[i] = s[4 + i] ? (const float *)s[4 + i]->data : nullptr;
+            a.x = (float *)n->data; a.x_stride = (int64_t)(n->nb[1] / 4);
+            if (n->ne[2] == 2) { a.h = (float *)((char *)n->data + n->nb[2]); a.h_stride = a.x_stride; }
+            a.n = n->ne[0]; a.n_tok = n->ne[1]; a.kind1 = n->op_params[2]; a.eps = ext_f(n, 3); a.kind2 = n->op_params[4]; a.y_scale = ext_f(n, 5);
+            B200_CHECK_RC(b200_op_norm_chain(&a, x.stream));
+            break;
+        }
+        case B200_EXT_TOKEN_SHIFT: {
+            b200_token_shift_args a;
+            memset(&a, 0, sizeof(a));
+            a.h = (const float *)s[0]->data; a.h_stride = (int64_t)(s[0]->nb[1] / 4);
+            a.mu = (const float *)s[1]->data; a.n_mix = (int32_t)n->ne[2]; a.width = (int32_t)n->ne[0]; a.n_tokens = (int32_t)n->ne[1];
+            a.seq_info = (const int32_t *)s[2]->data; a.n_seq = (int32_t)s[2]->ne[0];
+            a.prev = (float *)s[3]->data; a.slot_stride = (int64_t)(s[3]->nb[1] / 4);
+            a.dst = (float *)n->data; a.dst_s_tok = (int64_t)(n->nb[1] / 4); a.dst_s_mix = (int64_t)(n->nb[2] / 4);
+            B200_CHECK_RC(b200_op_token_shift(&a, x.stream));
+            break;
+        }
+        case B200_EXT_TIME_MIX_SCAN: {
+            b200_time_mix_args a;
+            memset(&a, 0, sizeof(a));
+            a.r = (const float *)s[0]->data; a.r_stride = (int64_t)(s[0]->nb[1] / 4);
+            a.k = (const float *)s[1]->data; a.k_stride = (int64_t)(s[1]->nb[1] / 4);
+            a.v = (const float *)s[2]->data; a.v_stride = (int64_t)(s[2]->nb[1] / 4);
+            a.z = (const float *)s[3]->data; a.z_stride = (int64_t)(s[3]->nb[1] / 4);
+            a.w0 = (const float *)s[4]->data; a.u = (const float *)s[5]->data;
+            a.seq_info = (const int32_t *)s[6]->data; a.n_seq = (int32_t)s[6]->ne[0];
+            a.state = (float *)s[7]->data; a.slot_stride = (int64_t)(s[7]->nb[1] / 4);
+            a.dst = (float *)n->data; a.dst_stride = (int64_t)(n->nb[1] / 4);
+            a.heads = n->op_params[2]; a.dim = n->op_params[3];
+            B200_CHECK_RC(b200_op_time_mix_scan(&a, x.stream));
+            break;
+        }
         default:
             backend_abort("graph_compute", "unknown extension op");
     }
@@ -447,6 +505,7 @@ bool op_supported(int /*device*/, const ggml_tensor *op) {
             return a == b && is_contiguous(s0) && is_contiguous(op);
         }
         case GGML_OP_GET_ROWS:
+            if (s0 && s0->type == GGML_TYPE_I32) return s1 && s1->type == GGML_TYPE_I32 && op->type == GGML_TYPE_I32;
             return s0 && s1 && s1->type == GGML_TYPE_I32 && op->type == GGML_TYPE_F32 &&
                    (s0->type == GGML_TYPE_F32 || s0->type == GGML_TYPE_F16 || is_hot_weight_type(s0->type));
         case GGML_OP_SOFT_MAX:

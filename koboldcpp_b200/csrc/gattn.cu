@@ -4,7 +4,7 @@
 // Cache rows are indexed by cell, one row per token holding all kv heads; which cells a token sees follows from the (sequence,
 // position) pairs of token and cell, so a batch may mix sequences, cells may be scattered, and a sliding window with kept first
 // positions needs no mask tensor.  The sink only enters the softmax denominator.  A table of score biases by distance (per head) may
-// join the scaled score, and the weights may be sigmoids of the scores instead of a softmax over them (nothing is normalised then).
+// join the scaled score (or a bias that grows linearly with the distance), and the weights may be sigmoids of the scores instead of a softmax over them (nothing is normalised then).
 #include "ops_util.cuh"
 #include <cuda_bf16.h>
 
@@ -13,7 +13,7 @@ using namespace opx;
 
 // ------------------------------------------------------------------------------------------------ bias + norm + rotation + cache store
 // One CTA per token.  The RMS statistics run over the whole projection (all heads at once) or, with norm_per_head, over every
-// head by itself (a warp per head, the scales parked in shared memory); q is rewritten in place, k and v go to the token's cache
+// head by itself (a warp per head, the scales parked in shared memory; with qk_unit_rms without a weight); q is rewritten in place, k and v go to the token's cache
 // rows.  A rotated pair is (2i, 2i + 1) or, with rope_halves, (i, i + n_dims / 2).
 __global__ void __launch_bounds__(1024) qkv_store_kernel(const b200_qkv_store_args a) {
     __shared__ float sh[32];
@@ -25,12 +25,12 @@ __global__ void __launch_bounds__(1024) qkv_store_kernel(const b200_qkv_store_ar
     const int64_t cell = a.cells[t];
     float *kc = a.k_cache + cell * a.k_cache_stride, *vc = a.v_cache + cell * a.v_cache_stride;
     float qs = 1.f, ks = 1.f;
-    const bool per_head = a.norm_per_head != 0;
+    const bool unit = a.qk_unit_rms != 0, per_head = a.norm_per_head != 0 || unit;
     if (per_head) {
         const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
         for (int hh = warp; hh < a.n_head + a.n_head_kv; hh += n_warps) {
             const bool is_k = hh >= a.n_head;
-            if (!(is_k ? a.k_norm : a.q_norm)) continue;  // warp-uniform
+            if (!unit && !(is_k ? a.k_norm : a.q_norm)) continue;  // warp-uniform
             const int e0 = (is_k ? hh - a.n_head : hh) * a.dim;
             const float *src = is_k ? k : q, *bias = is_k ? a.k_bias : a.q_bias;
             float s = 0.f;
@@ -60,20 +60,23 @@ __global__ void __launch_bounds__(1024) qkv_store_kernel(const b200_qkv_store_ar
         float *dst = which ? kc : q;
         const float *bias = which ? a.k_bias : a.q_bias, *nw = which ? a.k_norm : a.q_norm;
         const int heads = which ? a.n_head_kv : a.n_head;
+        if (!which && !unit && !nw && !bias && half == 0 && q_temp == 1.0f) continue;  // nothing changes q
         for (int idx = threadIdx.x; idx < heads * per_head_items; idx += blockDim.x) {
             const int hh = idx / per_head_items, j = idx - hh * per_head_items;
-            const float sc = (per_head && nw) ? head_scale[which * a.n_head + hh] : (which ? ks : qs);
+            const float sc = (per_head && (nw || unit)) ? head_scale[which * a.n_head + hh] : (which ? ks : qs);
             const int wb = per_head ? hh * a.dim : 0;  // the weight of entry e is nw[e - wb]
             if (j >= half) {
                 const int e = hh * a.dim + a.n_dims + (j - half);
                 float x = src[e] + (bias ? bias[e] : 0.f);
                 if (nw) x = x * sc * nw[e - wb];
+                else if (unit) x *= sc;
                 dst[e] = which ? x : x * q_temp;
                 continue;
             }
             const int e0 = hh * a.dim + (a.rope_halves ? j : 2 * j), e1 = a.rope_halves ? e0 + half : e0 + 1;
             float u = src[e0] + (bias ? bias[e0] : 0.f), w = src[e1] + (bias ? bias[e1] : 0.f);
             if (nw) { u = u * sc * nw[e0 - wb]; w = w * sc * nw[e1 - wb]; }
+            else if (unit) { u *= sc; w *= sc; }
             float sn, cs;
             sincosf(p * a.freqs[j], &sn, &cs);
             const float tq = which ? 1.0f : q_temp;
@@ -100,15 +103,20 @@ __device__ __forceinline__ bool sa_visible(int cell_seq, int cell_pos, int seq, 
     return cell_seq == seq && cell_pos <= pos && cell_pos >= lo && (window <= 0 || pos - cell_pos < window || cell_pos < keep_first);
 }
 __device__ __forceinline__ int sa_chunk_start(int pos, int chunk) { return chunk > 0 ? pos - pos % chunk : 0; }
-// the bias of a key `dist` positions behind the query (0 without a table)
-__device__ __forceinline__ float sa_dist_bias(const b200_sink_attn_args &a, int dist, int h) {
+// the bias of a key `dist` positions behind the query (0 without a table); lin: the head's bias per position of distance
+__device__ __forceinline__ float sa_dist_slope(const b200_sink_attn_args &a, int h) { return (a.dist_bias && a.dist_linear) ? a.dist_bias[(int64_t)h * a.n_dist] : 0.f; }
+__device__ __forceinline__ float sa_dist_bias(const b200_sink_attn_args &a, int dist, int h, float lin) {
+    if (a.dist_linear) return lin * (float)dist;
     return a.dist_bias ? a.dist_bias[(int64_t)h * a.n_dist + min(dist, a.n_dist - 1)] : 0.f;  // a head's row is contiguous: neighbouring keys share cache lines
 }
 __device__ __forceinline__ float sa_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 // for weights that are rounded to bf16 right away (8 bits of mantissa): the fast exponential and division are exact enough
 __device__ __forceinline__ float sa_sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
 __device__ __forceinline__ float sa_head_gate(const b200_sink_attn_args &a, int64_t t, int h) {
-    return a.gate ? 1.0f / (1.0f + expf(-a.gate[t * a.gate_stride + h])) : 1.0f;
+    return ((a.gate && !a.gate_per_value) ? 1.0f / (1.0f + expf(-a.gate[t * a.gate_stride + h])) : 1.0f) * a.out_scale;
+}
+__device__ __forceinline__ float sa_value_gate(const b200_sink_attn_args &a, int64_t t, int h, int j) {
+    return (a.gate && a.gate_per_value) ? 1.0f / (1.0f + expf(-a.gate[t * a.gate_stride + (int64_t)h * a.vdim + j])) : 1.0f;
 }
 
 // ------------------------------------------------------------------------------------------------ attention, f32 products
@@ -136,6 +144,7 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attn_kernel(const b200_sink_a
     const int seq = a.tok_seq[t], pos = a.tok_pos[t], lo = sa_chunk_start(pos, a.chunk);
     const bool sig = a.weights == B200_ATTN_SIGMOID;
     float m = sig ? 0.f : -INFINITY, l = 0.f;  // sigmoid weights: no maximum, no sum; the warps' accumulators simply add up
+    const float lin = sa_dist_slope(a, h);
     const int per_split = ((a.n_kv + n_split - 1) / n_split + 31) & ~31;
     const int c_begin = (int)blockIdx.z * per_split, c_end = min(a.n_kv, c_begin + per_split);
     for (int cb = c_begin + warp * 32; cb < c_end; cb += WARPS * 32) {
@@ -146,7 +155,7 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attn_kernel(const b200_sink_a
             mine = sa_visible(a.cell_seq[cb + lane], cp, seq, pos, a.window, a.keep_first, lo);
             my_dist = pos - cp;
         }
-        const float my_bias = mine ? sa_dist_bias(a, my_dist, h) : 0.f;  // lane j holds the bias of cell cb + j
+        const float my_bias = mine ? sa_dist_bias(a, my_dist, h, lin) : 0.f;  // lane j holds the bias of cell cb + j
         unsigned rest = __ballot_sync(0xffffffffu, mine);
         while (rest) {
             bool vis[SA_UNROLL];  // warp-uniform
@@ -224,7 +233,7 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attn_kernel(const b200_sink_a
     for (int j = threadIdx.x; j < V; j += blockDim.x) {
         float o = 0.f;
         for (int w = 0; w < WARPS; w++) o += smem[(size_t)w * V + j] * sl[w];
-        out[j] = o * inv;
+        out[j] = o * inv * sa_value_gate(a, t, h, j);
     }
 }
 
@@ -245,7 +254,7 @@ __global__ void __launch_bounds__(128) sink_attn_merge_kernel(const b200_sink_at
     for (int j = threadIdx.x; j < V; j += blockDim.x) {
         float o = 0.f;
         for (int z = 0; z < n_split; z++) { const float mz = pp[(int64_t)z * (V + 2)]; if (mz != -INFINITY) o += pp[(int64_t)z * (V + 2) + 2 + j] * expf(mz - M); }
-        out[j] = o * inv;
+        out[j] = o * inv * sa_value_gate(a, t, h, j);
     }
 }
 
@@ -379,6 +388,7 @@ __global__ void __launch_bounds__(GM_WARPS * 32) sink_attn_mma_kernel(const b200
     for (int j = 0; j < 2 * VS; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // rows g and g + 8; l: this lane's share of the row sum
     const bool sig = a.weights == B200_ATTN_SIGMOID;
+    const float lin = sa_dist_slope(a, h);
 
     for (int c0 = 0; c0 < a.n_kv; c0 += GM_CELLS) {
         // does any of the warp's tokens see any of the tile's cells?  lane = cell
@@ -419,8 +429,8 @@ __global__ void __launch_bounds__(GM_WARPS * 32) sink_attn_mma_kernel(const b200
             for (int e = 0; e < 2; e++) {
                 const int c = j * 8 + 2 * t4 + e;
                 const int xs = cseq[c], xp = cpos[c];
-                s[j][e] = sa_visible(xs, xp, rs0, rp0, a.window, a.keep_first, rl0) ? s[j][e] * a.scale + sa_dist_bias(a, rp0 - xp, h) : -INFINITY;
-                s[j][2 + e] = sa_visible(xs, xp, rs1, rp1, a.window, a.keep_first, rl1) ? s[j][2 + e] * a.scale + sa_dist_bias(a, rp1 - xp, h) : -INFINITY;
+                s[j][e] = sa_visible(xs, xp, rs0, rp0, a.window, a.keep_first, rl0) ? s[j][e] * a.scale + sa_dist_bias(a, rp0 - xp, h, lin) : -INFINITY;
+                s[j][2 + e] = sa_visible(xs, xp, rs1, rp1, a.window, a.keep_first, rl1) ? s[j][2 + e] * a.scale + sa_dist_bias(a, rp1 - xp, h, lin) : -INFINITY;
                 mx0 = fmaxf(mx0, s[j][e]); mx1 = fmaxf(mx1, s[j][2 + e]);
             }
         }
@@ -496,8 +506,8 @@ __global__ void __launch_bounds__(GM_WARPS * 32) sink_attn_mma_kernel(const b200
 #pragma unroll
         for (int j = 0; j < 2 * VS; j++) {
             const int c = 8 * j + 2 * t4;
-            if (c < V) out[c] = o[j][2 * hh] * w[hh];
-            if (c + 1 < V) out[c + 1] = o[j][2 * hh + 1] * w[hh];
+            if (c < V) out[c] = o[j][2 * hh] * w[hh] * sa_value_gate(a, t, h, c);
+            if (c + 1 < V) out[c + 1] = o[j][2 * hh + 1] * w[hh] * sa_value_gate(a, t, h, c + 1);
         }
     }
 }
@@ -578,10 +588,23 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
         const int nt = min(LA_CHUNK, count - t0);
         __syncthreads();  // the previous chunk has been read
 #pragma unroll
-        for (int j = 0; j < NQ; j++) { sq[tid + j * LA_WARPS * 32] = la_act(pq[j], a.act); sk[tid + j * LA_WARPS * 32] = la_act(pk[j], a.act); }
+        for (int j = 0; j < NQ; j++) { sq[tid + j * LA_WARPS * 32] = la_act(pq[j], a.act); sk[tid + j * LA_WARPS * 32] = la_act(pk[j], a.act) * a.k_scale; }
 #pragma unroll
         for (int j = 0; j < NVV; j++) sv[tid + j * LA_WARPS * 32] = la_act(pv[j], a.act);
         __syncthreads();
+        if (a.n_dims > 0) {  // rotation of entry i with entry i + n_dims / 2 where the rows wait (the scale on k commutes with it)
+            const int half = a.n_dims / 2;
+            for (int idx = tid; idx < nt * half; idx += LA_WARPS * 32) {
+                const int tt = idx / half, i = idx - tt * half;
+                float sn, cs;
+                sincosf((float)a.pos[first + t0 + tt] * a.freqs[i], &sn, &cs);
+                float *pq0 = sq + tt * DP + i, *pk0 = sk + tt * DP + i;
+                const float qu = pq0[0], qw = pq0[half], ku = pk0[0], kw = pk0[half];
+                pq0[0] = qu * cs - qw * sn; pq0[half] = qw * cs + qu * sn;
+                pk0[0] = ku * cs - kw * sn; pk0[half] = kw * cs + ku * sn;
+            }
+            __syncthreads();
+        }
         if (t0 + LA_CHUNK < count) fetch(t0 + LA_CHUNK);
         for (int tt0 = 0; tt0 < nt; tt0 += LA_RG) {
             // the row sums do not feed the recurrence: LA_RG tokens x LA_CW columns = 32 partial sums per lane are added up across
@@ -649,7 +672,7 @@ extern "C" int b200_op_qkv_store(const b200_qkv_store_args *a, b200_stream_t str
     if (a->n_tokens == 0) return B200_OK;
     // few tokens (decode): a token's row is all the parallelism there is, so its CTA is wide
     const int threads = a->n_tokens <= 64 ? 1024 : 256;
-    const size_t smem = a->norm_per_head ? (size_t)(a->n_head + a->n_head_kv) * sizeof(float) : 0;
+    const size_t smem = (a->norm_per_head || a->qk_unit_rms) ? (size_t)(a->n_head + a->n_head_kv) * sizeof(float) : 0;
     OPX_REQUIRE(smem <= 32 * 1024, B200_ERR_UNSUPPORTED, "b200_op_qkv_store: per-head norms over at most 8192 heads");
     qkv_store_kernel<<<(unsigned)a->n_tokens, threads, smem, (cudaStream_t)stream>>>(*a);
     B200_CUDA_TRY(cudaGetLastError());
@@ -665,8 +688,12 @@ extern "C" size_t b200_sink_attn_workspace_bytes(const b200_sink_attn_args *a) {
 
 extern "C" int b200_op_sink_attn(const b200_sink_attn_args *a, b200_stream_t stream) { return b200_op_sink_attn_ws(a, nullptr, 0, stream); }
 
-extern "C" int b200_op_sink_attn_ws(const b200_sink_attn_args *a, void *workspace, size_t workspace_bytes, b200_stream_t stream) {
-    OPX_REQUIRE(a && a->q && a->k_cache && a->v_cache && a->cell_seq && a->cell_pos && a->tok_seq && a->tok_pos && a->dst, B200_ERR_INVALID, "b200_op_sink_attn: NULL argument");
+extern "C" int b200_op_sink_attn_ws(const b200_sink_attn_args *args, void *workspace, size_t workspace_bytes, b200_stream_t stream) {
+    OPX_REQUIRE(args, B200_ERR_INVALID, "b200_op_sink_attn: NULL argument");
+    b200_sink_attn_args copy = *args;
+    if (copy.out_scale == 0.0f) copy.out_scale = 1.0f;
+    const b200_sink_attn_args *a = &copy;
+    OPX_REQUIRE(a->q && a->k_cache && a->v_cache && a->cell_seq && a->cell_pos && a->tok_seq && a->tok_pos && a->dst, B200_ERR_INVALID, "b200_op_sink_attn: NULL argument");
     OPX_REQUIRE(a->n_head > 0 && a->n_head <= 65535 && a->n_head_kv > 0 && a->n_head % a->n_head_kv == 0 && a->dim > 0 && a->dim <= 256 && a->vdim > 0 && a->vdim <= 256 &&
                 a->n_tokens >= 0 && a->n_kv >= 0 && a->window >= 0 && a->keep_first >= 0 && a->chunk >= 0, B200_ERR_UNSUPPORTED, "b200_op_sink_attn: head sizes up to 256, heads up to 65535");
     OPX_REQUIRE((a->weights == B200_ATTN_SOFTMAX || a->weights == B200_ATTN_SIGMOID) && (!a->dist_bias || a->n_dist > 0), B200_ERR_INVALID, "b200_op_sink_attn: weight kind / distance table");
@@ -683,8 +710,13 @@ extern "C" int b200_op_sink_attn_ws(const b200_sink_attn_args *a, void *workspac
     return launch_sink_attn<8>(a, part, n_split, st);
 }
 
-extern "C" int b200_op_linear_attn_scan(const b200_linear_attn_args *a, b200_stream_t stream) {
-    OPX_REQUIRE(a && a->q && a->k && a->v && a->decay && a->seq_info && a->state && a->dst, B200_ERR_INVALID, "b200_op_linear_attn_scan: NULL argument");
+extern "C" int b200_op_linear_attn_scan(const b200_linear_attn_args *args, b200_stream_t stream) {
+    OPX_REQUIRE(args, B200_ERR_INVALID, "b200_op_linear_attn_scan: NULL argument");
+    b200_linear_attn_args copy = *args;
+    if (copy.k_scale == 0.0f) copy.k_scale = 1.0f;
+    const b200_linear_attn_args *a = &copy;
+    OPX_REQUIRE(a->n_dims == 0 || (a->n_dims > 0 && a->n_dims % 2 == 0 && a->n_dims <= a->dim && a->pos && a->freqs), B200_ERR_INVALID, "b200_op_linear_attn_scan: rotation does not fit dim");
+    OPX_REQUIRE(a->q && a->k && a->v && a->decay && a->seq_info && a->state && a->dst, B200_ERR_INVALID, "b200_op_linear_attn_scan: NULL argument");
     OPX_REQUIRE(a->heads > 0 && a->heads <= 65535 && a->dim > 0 && a->dim <= 256 && a->vdim > 0 && a->n_seq >= 0 && a->n_seq <= 65535 &&
                 a->slot_stride >= (int64_t)a->heads * a->dim * a->vdim, B200_ERR_UNSUPPORTED, "b200_op_linear_attn_scan: dim up to 256");
     if (a->n_seq == 0) return B200_OK;

@@ -264,6 +264,7 @@ const Arch *genesun_arch();
 const Arch *galirax_arch();
 const Arch *zevopel_arch();
 const Arch *medodra_arch();
+const Arch *mafuzen_arch();
 
 }  // namespace host
 }  // namespace b200

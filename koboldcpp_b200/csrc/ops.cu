@@ -175,6 +175,7 @@ __device__ __forceinline__ float unary_apply(int op, float x, float p0, float p1
         case B200_UN_SCALE: return x * p0;
         case B200_UN_CLAMP: return x < p0 ? p0 : (x > p1 ? p1 : x);
         case B200_UN_SOFTCAP: return p0 * tanhf(x / p0);
+        case B200_UN_RELU_SQR: { const float r = fmaxf(x, 0.f); return r * r; }
     }
     return x;
 }
@@ -932,7 +933,7 @@ extern "C" int b200_op_unary(int op, const b200_tensor *x, const b200_tensor *ds
     REQUIRE(x && dst && x->data && dst->data, B200_ERR_INVALID, "b200_op_unary: NULL argument");
     REQUIRE(x->type == B200_TYPE_F32 && dst->type == B200_TYPE_F32 && contiguous(x) && contiguous(dst) && nelements(x) == nelements(dst),
             B200_ERR_UNSUPPORTED, "b200_op_unary: contiguous f32 only");
-    REQUIRE(op >= 0 && op <= B200_UN_SOFTCAP, B200_ERR_INVALID, "b200_op_unary: bad op %d", op);
+    REQUIRE(op >= 0 && op <= B200_UN_RELU_SQR, B200_ERR_INVALID, "b200_op_unary: bad op %d", op);
     const int64_t n = nelements(x);
     if (n == 0) return B200_OK;
     unary_kernel<<<grid1d(n, 256), 256, 0, (cudaStream_t)stream>>>(op, (const float *)x->data, (float *)dst->data, n, p0, p1);
@@ -1058,8 +1059,9 @@ extern "C" int b200_op_cpy_indirect(const b200_tensor *src, const b200_tensor *d
 
 extern "C" int b200_op_get_rows(const b200_tensor *src, const b200_tensor *ids, const b200_tensor *dst, b200_stream_t stream) {
     REQUIRE(src && ids && dst && src->data && ids->data && dst->data, B200_ERR_INVALID, "b200_op_get_rows: NULL argument");
-    REQUIRE(ids->type == B200_TYPE_I32 && dst->type == B200_TYPE_F32 && dst->nb[0] == 4, B200_ERR_UNSUPPORTED, "b200_op_get_rows: i32 ids, f32 dst");
-    const int t = src->type;
+    REQUIRE(ids->type == B200_TYPE_I32 && dst->type == (src->type == B200_TYPE_I32 ? B200_TYPE_I32 : B200_TYPE_F32) && dst->nb[0] == 4, B200_ERR_UNSUPPORTED,
+            "b200_op_get_rows: i32 ids, f32 dst (i32 for an i32 table)");
+    const int t = src->type == B200_TYPE_I32 ? B200_TYPE_F32 : src->type;  // integers are copied as the 32-bit words they are
     REQUIRE(t == B200_TYPE_F32 || t == B200_TYPE_F16 || t == B200_TYPE_Q4_0 || t == B200_TYPE_Q8_0 || t == B200_TYPE_Q4_K || t == B200_TYPE_Q5_K || t == B200_TYPE_Q6_K ||
             t == B200_TYPE_Q4_1 || t == B200_TYPE_Q5_0 || t == B200_TYPE_Q5_1 || t == B200_TYPE_Q2_K || t == B200_TYPE_Q3_K ||
             t == B200_TYPE_IQ4_NL || t == B200_TYPE_IQ4_XS,

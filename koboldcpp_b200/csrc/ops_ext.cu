@@ -225,6 +225,75 @@ __global__ void __launch_bounds__(1024) norm_pair_kernel(TD x1, const float *__r
     }
 }
 
+// A sublayer's result (or the weighted sum over a token's experts and a shared one) behind its norm, the residual stream, and the
+// input norm of the next sublayer: one CTA per token, the row in registers throughout.  Everything a thread reads -- result rows,
+// residual, both norms' vectors -- is requested before the first block-wide sum (rows longer than 8 values per thread fetch the
+// second norm's vectors where they are used: registers).
+template <int VPT>
+__global__ void __launch_bounds__(1024) norm_chain_kernel(const b200_norm_chain_args a) {
+    constexpr bool EARLY = VPT <= 4;
+    __shared__ float sh[32];
+    const int64_t t = blockIdx.x;
+    const int n = (int)a.n;
+    float v[VPT], w1[VPT], b1[VPT], w2[VPT], b2[VPT], rv[VPT];
+#pragma unroll
+    for (int k = 0; k < VPT; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        const bool ok = i < n;
+        v[k] = 0.f;
+        w1[k] = (a.w1 && ok) ? a.w1[i] : 1.f;
+        b1[k] = (a.b1 && ok) ? a.b1[i] : 0.f;
+        rv[k] = (a.res && ok) ? a.res[t * a.res_stride + i] : 0.f;
+        if (EARLY && a.h) { w2[k] = (a.w2 && ok) ? a.w2[i] : 1.f; b2[k] = (a.b2 && ok) ? a.b2[i] : 0.f; }
+    }
+    for (int kk = 0; kk < a.n_y; kk++) {
+        const float wk = a.yw ? a.yw[t * a.yw_s_tok + kk] : 1.0f;
+        const float *yk = a.y + t * a.y_s_tok + kk * a.y_s_slot;
+#pragma unroll
+        for (int k = 0; k < VPT; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i < n) v[k] += wk * yk[i];
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < VPT; k++) {
+        const int i = threadIdx.x + k * blockDim.x;
+        v[k] *= a.y_scale;
+        if (a.shared && i < n) v[k] += a.shared[t * a.shared_stride + i];
+    }
+#pragma unroll
+    for (int pass = 0; pass < 2; pass++) {
+        if (pass == 1 && !a.h) break;
+        const int kind = pass ? a.kind2 : a.kind1;
+        float mean = 0.f, ss = 0.f;
+        if (kind == B200_NORM_LAYER) {
+            float s = 0.f;
+#pragma unroll
+            for (int k = 0; k < VPT; k++) s += v[k];  // values beyond the row are zero
+            mean = block_sum(s, sh) / (float)n;
+        }
+#pragma unroll
+        for (int k = 0; k < VPT; k++) { const float d = threadIdx.x + k * blockDim.x < n ? v[k] - mean : 0.f; ss += d * d; }
+        const float scale = 1.0f / sqrtf(block_sum(ss, sh) / (float)n + a.eps);
+        if (pass == 0) {
+#pragma unroll
+            for (int k = 0; k < VPT; k++) {
+                const int i = threadIdx.x + k * blockDim.x;
+                v[k] = i < n ? rv[k] + ((v[k] - mean) * scale * w1[k] + b1[k]) : 0.f;
+                if (i < n) a.x[t * a.x_stride + i] = v[k];
+            }
+        } else {
+#pragma unroll
+            for (int k = 0; k < VPT; k++) {
+                const int i = threadIdx.x + k * blockDim.x;
+                if (i >= n) continue;
+                const float w = EARLY ? w2[k] : (a.w2 ? a.w2[i] : 1.f), b = EARLY ? b2[k] : (a.b2 ? a.b2[i] : 0.f);
+                a.h[t * a.h_stride + i] = (v[k] - mean) * scale * w + b;
+            }
+        }
+    }
+}
+
 // position vector of sines and cosines added to every row: a thread per pair (2i, 2i + 1), the angle pos * f_i in f32
 __global__ void add_sinusoid_kernel(TD x, const int32_t *__restrict__ pos, const float *__restrict__ freqs, TD dst, int64_t pairs, int64_t total) {
     const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -255,6 +324,23 @@ extern "C" int b200_op_norm_pair(const b200_tensor *x1, const float *w1, const f
 #define B200_NP(V) norm_pair_kernel<V><<<(unsigned)rows, rb, 0, (cudaStream_t)stream>>>(td(x1), w1, b1, td(x2), w2, td(dst), eps)
     if (vpt <= 4) B200_NP(4); else if (vpt <= 8) B200_NP(8); else B200_NP(16);
 #undef B200_NP
+    B200_CUDA_TRY(cudaGetLastError());
+    return B200_OK;
+}
+
+extern "C" int b200_op_norm_chain(const b200_norm_chain_args *args, b200_stream_t stream) {
+    OPX_REQUIRE(args && args->y && args->x, B200_ERR_INVALID, "b200_op_norm_chain: NULL argument");
+    b200_norm_chain_args a = *args;
+    if (a.y_scale == 0.0f) a.y_scale = 1.0f;
+    OPX_REQUIRE(a.n >= 0 && a.n <= 16384 && a.n_y >= 1 && a.n_tok >= 0, B200_ERR_UNSUPPORTED, "b200_op_norm_chain: rows of at most 16384 values, at least one result per token");
+    OPX_REQUIRE((a.kind1 == B200_NORM_LAYER || a.kind1 == B200_NORM_RMS) && (!a.h || a.kind2 == B200_NORM_LAYER || a.kind2 == B200_NORM_RMS), B200_ERR_INVALID, "b200_op_norm_chain: norm kind");
+    if (a.n == 0 || a.n_tok == 0) return B200_OK;
+    const int n = (int)a.n;
+    const int rb = n <= 256 ? 64 : n <= 512 ? 128 : n <= 1024 ? 256 : n <= 2048 ? 512 : 1024, vpt = (n + rb - 1) / rb;
+    const cudaStream_t st = (cudaStream_t)stream;
+    if (vpt <= 4) norm_chain_kernel<4><<<(unsigned)a.n_tok, rb, 0, st>>>(a);
+    else if (vpt <= 8) norm_chain_kernel<8><<<(unsigned)a.n_tok, rb, 0, st>>>(a);
+    else norm_chain_kernel<16><<<(unsigned)a.n_tok, rb, 0, st>>>(a);
     B200_CUDA_TRY(cudaGetLastError());
     return B200_OK;
 }

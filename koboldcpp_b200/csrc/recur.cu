@@ -1,5 +1,5 @@
 // recur.cu -- mixers that carry a fixed-size state per sequence instead of a cache row per token (include/b200_ggml_ops.h:
-// b200_op_short_conv, b200_op_delta_rule_scan, b200_op_mingru_scan).  A batch names its sequences through seq_info (first token,
+// b200_op_short_conv, b200_op_delta_rule_scan, b200_op_mingru_scan, b200_op_token_shift, b200_op_time_mix_scan).  A batch names its sequences through seq_info (first token,
 // token count, state slot, fresh); a fresh sequence starts from zeros whatever its slot held before.  Everything is f32.
 #include "ops_util.cuh"
 
@@ -256,9 +256,169 @@ __global__ void __launch_bounds__(32 * MG_SEG_MAX) mingru_scan_kernel(const b200
     if (seg == 0 && live) *Sp = sS[lane];
 }
 
+// ------------------------------------------------------------------------------------------------ token shift
+// A thread per channel, a CTA per (128 channels, TS_TOK tokens of one sequence): the TS_TOK + 1 inputs travel to registers at once and
+// serve all mixes.  Only the CTA of a portion's first tokens reads the slot, and it alone rewrites it (thread = channel).
+constexpr int TS_TOK = 16;
+__global__ void __launch_bounds__(128) token_shift_kernel(const b200_token_shift_args a) {
+    const int c = blockIdx.x * 128 + threadIdx.x, s = blockIdx.z;
+    const int first = a.seq_info[s], count = a.seq_info[a.n_seq + s], slot = a.seq_info[2 * a.n_seq + s], fresh = a.seq_info[3 * a.n_seq + s];
+    const int t0 = blockIdx.y * TS_TOK;
+    if (c >= a.width || t0 >= count) return;
+    const int nt = min(TS_TOK, count - t0);
+    float *prev = a.prev + (int64_t)slot * a.slot_stride + c;
+    float win[TS_TOK + 1];
+    win[0] = t0 > 0 ? a.h[(int64_t)(first + t0 - 1) * a.h_stride + c] : (fresh ? 0.f : *prev);
+#pragma unroll
+    for (int i = 0; i < TS_TOK; i++) win[i + 1] = i < nt ? a.h[(int64_t)(first + t0 + i) * a.h_stride + c] : 0.f;
+    if (t0 == 0) *prev = a.h[(int64_t)(first + count - 1) * a.h_stride + c];
+    for (int m = 0; m < a.n_mix; m++) {
+        const float mu = a.mu[(int64_t)m * a.width + c];
+        float *dst = a.dst + (int64_t)m * a.dst_s_mix + (int64_t)(first + t0) * a.dst_s_tok + c;
+#pragma unroll
+        for (int i = 0; i < TS_TOK; i++) if (i < nt) dst[(int64_t)i * a.dst_s_tok] = win[i + 1] + (win[i] - win[i + 1]) * mu;
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ time mixing
+// The columns of the state never interact: a warp owns TM_CW columns of one (sequence, head) and keeps them in registers over the
+// whole token loop, a lane the key channels d = lane, lane + 32, ...  Column j sees  o_j = sum_d r_d S_dj + (sum_d r_d u_d k_d) v_j
+// and  S_dj <- w_d S_dj + k_d v_j;  the bracket is the same for every column, so a lane adds its share of it once per token.  The
+// inputs of CHUNK tokens are staged in shared memory (decays computed there once per CTA) while the next chunk travels to registers.
+// The read-outs do not feed the recurrence: 8 tokens x 4 columns of partial sums per lane are added up across the warp in one
+// halving exchange.
+constexpr int TM_CW = 4, TM_WARPS = 4, TM_COLS = TM_CW * TM_WARPS, TM_RG = 8;
+static_assert(TM_RG * TM_CW == 32 && TM_CW == 4, "one partial sum per lane");
+template <int DPL>
+__global__ void __launch_bounds__(TM_WARPS * 32) time_mix_scan_kernel(const b200_time_mix_args a) {
+    constexpr int CHUNK = DPL <= 4 ? 16 : 8, DP = 32 * DPL, NT = TM_WARPS * 32;
+    __shared__ float sr[CHUNK * DP], sk[CHUNK * DP], sw[CHUNK * DP], sv[CHUNK * TM_COLS];
+    const int h = blockIdx.y, s = blockIdx.z;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
+    const int D = a.dim;
+    const int first = a.seq_info[s], count = a.seq_info[a.n_seq + s], slot = a.seq_info[2 * a.n_seq + s], fresh = a.seq_info[3 * a.n_seq + s];
+    if (count <= 0) return;
+    const int cb = blockIdx.x * TM_COLS, col0 = cb + warp * TM_CW;
+    float *Sp = a.state + (int64_t)slot * a.slot_stride + ((int64_t)h * D + col0) * D;
+    float S[TM_CW][DPL], u[DPL];
+#pragma unroll
+    for (int i = 0; i < DPL; i++) {
+        const int d = lane + 32 * i;
+        u[i] = d < D ? a.u[h * D + d] : 0.f;
+#pragma unroll
+        for (int c = 0; c < TM_CW; c++) S[c][i] = (!fresh && d < D && col0 + c < D) ? Sp[(int64_t)c * D + d] : 0.f;
+    }
+    constexpr int NQ = CHUNK * DP / NT, NV = CHUNK * TM_COLS / NT;
+    float pr[NQ], pk[NQ], pz[NQ], pv[NV];
+    auto fetch = [&](int t0) {
+        const int nt = min(CHUNK, count - t0);
+#pragma unroll
+        for (int j = 0; j < NQ; j++) {
+            const int idx = tid + j * NT, tt = idx / DP, d = idx - tt * DP;
+            const bool ok = tt < nt && d < D;
+            const int64_t tok = first + t0 + tt;
+            pr[j] = ok ? a.r[tok * a.r_stride + (int64_t)h * D + d] : 0.f;
+            pk[j] = ok ? a.k[tok * a.k_stride + (int64_t)h * D + d] : 0.f;
+            pz[j] = ok ? a.z[tok * a.z_stride + (int64_t)h * D + d] + a.w0[h * D + d] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < NV; j++) {
+            const int idx = tid + j * NT, tt = idx / TM_COLS, c = idx - tt * TM_COLS;
+            pv[j] = (tt < nt && cb + c < D) ? a.v[(int64_t)(first + t0 + tt) * a.v_stride + (int64_t)h * D + cb + c] : 0.f;
+        }
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < count; t0 += CHUNK) {
+        const int nt = min(CHUNK, count - t0);
+        __syncthreads();  // the previous chunk has been read
+#pragma unroll
+        for (int j = 0; j < NQ; j++) { sr[tid + j * NT] = pr[j]; sk[tid + j * NT] = pk[j]; sw[tid + j * NT] = expf(-expf(pz[j])); }
+#pragma unroll
+        for (int j = 0; j < NV; j++) sv[tid + j * NT] = pv[j];
+        __syncthreads();
+        if (t0 + CHUNK < count) fetch(t0 + CHUNK);
+        for (int tt0 = 0; tt0 < nt; tt0 += TM_RG) {
+            float part[TM_RG * TM_CW];
+#pragma unroll
+            for (int g = 0; g < TM_RG; g++) {
+                const int tt = tt0 + g;
+                if (tt < nt) {  // warp-uniform
+                    float rv[DPL], kv[DPL], wv[DPL], bonus = 0.f;
+#pragma unroll
+                    for (int i = 0; i < DPL; i++) {
+                        const int d = tt * DP + lane + 32 * i;
+                        rv[i] = sr[d]; kv[i] = sk[d]; wv[i] = sw[d];
+                        bonus += rv[i] * (u[i] * kv[i]);
+                    }
+#pragma unroll
+                    for (int c = 0; c < TM_CW; c++) {
+                        const float vc = sv[tt * TM_COLS + warp * TM_CW + c];
+                        float acc = bonus * vc;
+#pragma unroll
+                        for (int i = 0; i < DPL; i++) { acc += S[c][i] * rv[i]; S[c][i] = wv[i] * S[c][i] + kv[i] * vc; }
+                        part[g * TM_CW + c] = acc;
+                    }
+                } else {
+#pragma unroll
+                    for (int c = 0; c < TM_CW; c++) part[g * TM_CW + c] = 0.f;
+                }
+            }
+#pragma unroll
+            for (int off = 16, n = 32; off >= 1; off >>= 1, n >>= 1) {
+                const bool upper = (lane & off) != 0;
+#pragma unroll
+                for (int i = 0; i < n / 2; i++) {
+                    const float send = upper ? part[i] : part[i + n / 2], keep = upper ? part[i + n / 2] : part[i];
+                    part[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+                }
+            }
+            const int tt = tt0 + (lane >> 2), c = lane & 3;  // TM_CW == 4
+            if (tt < nt && col0 + c < D) a.dst[(int64_t)(first + t0 + tt) * a.dst_stride + (int64_t)h * D + col0 + c] = part[0];
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < DPL; i++) {
+        const int d = lane + 32 * i;
+#pragma unroll
+        for (int c = 0; c < TM_CW; c++) if (d < D && col0 + c < D) Sp[(int64_t)c * D + d] = S[c][i];
+    }
+}
+
+template <int DPL>
+static int launch_time_mix(const b200_time_mix_args *a, cudaStream_t st) {
+    const dim3 grid((unsigned)((a->dim + TM_COLS - 1) / TM_COLS), (unsigned)a->heads, (unsigned)a->n_seq);
+    time_mix_scan_kernel<DPL><<<grid, TM_WARPS * 32, 0, st>>>(*a);
+    B200_CUDA_TRY(cudaGetLastError());
+    return B200_OK;
+}
+
 }  // namespace b200
 
 using namespace b200;
+
+extern "C" int b200_op_token_shift(const b200_token_shift_args *a, b200_stream_t stream) {
+    OPX_REQUIRE(a && a->h && a->mu && a->seq_info && a->prev && a->dst, B200_ERR_INVALID, "b200_op_token_shift: NULL argument");
+    OPX_REQUIRE(a->width > 0 && a->n_mix > 0 && a->n_seq >= 0 && a->n_seq <= 65535 && a->n_tokens >= 0 && a->n_tokens <= 65535 * TS_TOK && a->slot_stride >= a->width, B200_ERR_INVALID,
+                "b200_op_token_shift: bad sizes");
+    if (a->n_seq == 0 || a->n_tokens == 0) return B200_OK;
+    const dim3 grid((unsigned)((a->width + 127) / 128), (unsigned)((a->n_tokens + TS_TOK - 1) / TS_TOK), (unsigned)a->n_seq);
+    token_shift_kernel<<<grid, 128, 0, (cudaStream_t)stream>>>(*a);
+    B200_CUDA_TRY(cudaGetLastError());
+    return B200_OK;
+}
+
+extern "C" int b200_op_time_mix_scan(const b200_time_mix_args *a, b200_stream_t stream) {
+    OPX_REQUIRE(a && a->r && a->k && a->v && a->z && a->w0 && a->u && a->seq_info && a->state && a->dst, B200_ERR_INVALID, "b200_op_time_mix_scan: NULL argument");
+    OPX_REQUIRE(a->heads > 0 && a->heads <= 65535 && a->dim > 0 && a->dim <= 256 && a->n_seq >= 0 && a->n_seq <= 65535 && a->slot_stride >= (int64_t)a->heads * a->dim * a->dim,
+                B200_ERR_UNSUPPORTED, "b200_op_time_mix_scan: dim up to 256");
+    if (a->n_seq == 0) return B200_OK;
+    const cudaStream_t st = (cudaStream_t)stream;
+    const int dpl = (a->dim + 31) / 32;
+    if (dpl <= 1) return launch_time_mix<1>(a, st);
+    if (dpl <= 2) return launch_time_mix<2>(a, st);
+    if (dpl <= 4) return launch_time_mix<4>(a, st);
+    return launch_time_mix<8>(a, st);
+}
 
 extern "C" int b200_op_short_conv(const b200_short_conv_args *a, b200_stream_t stream) {
     OPX_REQUIRE(a && a->x && a->w && a->seq_info && a->dst && (a->tail || a->taps <= 1), B200_ERR_INVALID, "b200_op_short_conv: NULL argument");

@@ -88,7 +88,7 @@ class QkvStoreArgs(C.Structure):
                 ("pos", C.c_void_p), ("cells", C.c_void_p), ("freqs", C.c_void_p), ("k_cache", C.c_void_p), ("k_cache_stride", C.c_int64),
                 ("v_cache", C.c_void_p), ("v_cache_stride", C.c_int64), ("n_head", C.c_int32), ("n_head_kv", C.c_int32), ("dim", C.c_int32),
                 ("vdim", C.c_int32), ("n_dims", C.c_int32), ("n_tokens", C.c_int32), ("eps", C.c_float), ("norm_per_head", C.c_int32), ("rope_halves", C.c_int32),
-                ("v_unit_rms", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32)]
+                ("v_unit_rms", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32), ("qk_unit_rms", C.c_int32)]
 
 
 class SinkAttnArgs(C.Structure):
@@ -98,14 +98,16 @@ class SinkAttnArgs(C.Structure):
                 ("sink", C.c_void_p), ("dst", C.c_void_p), ("dst_stride", C.c_int64), ("n_head", C.c_int32), ("n_head_kv", C.c_int32), ("dim", C.c_int32),
                 ("vdim", C.c_int32), ("n_tokens", C.c_int32), ("n_kv", C.c_int32), ("window", C.c_int32), ("keep_first", C.c_int32), ("scale", C.c_float),
                 ("bf16_products", C.c_int32), ("chunk", C.c_int32), ("gate", C.c_void_p), ("gate_stride", C.c_int64),
-                ("weights", C.c_int32), ("dist_bias", C.c_void_p), ("n_dist", C.c_int32)]
+                ("weights", C.c_int32), ("dist_bias", C.c_void_p), ("n_dist", C.c_int32), ("dist_linear", C.c_int32), ("gate_per_value", C.c_int32),
+                ("out_scale", C.c_float)]
 
 
 class LinearAttnArgs(C.Structure):
     """b200_linear_attn_args (include/b200_ggml_ops.h); strides in floats."""
     _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("q_stride", C.c_int64), ("k_stride", C.c_int64), ("v_stride", C.c_int64),
                 ("decay", C.c_void_p), ("seq_info", C.c_void_p), ("n_seq", C.c_int32), ("state", C.c_void_p), ("slot_stride", C.c_int64),
-                ("dst", C.c_void_p), ("dst_stride", C.c_int64), ("heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("act", C.c_int32)]
+                ("dst", C.c_void_p), ("dst_stride", C.c_int64), ("heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("act", C.c_int32), ("k_scale", C.c_float),
+                ("pos", C.c_void_p), ("freqs", C.c_void_p), ("n_dims", C.c_int32)]
 
 
 class ShortConvArgs(C.Structure):
@@ -129,6 +131,27 @@ class MinGruArgs(C.Structure):
     _fields_ = [("z", C.c_void_p), ("x", C.c_void_p), ("g", C.c_void_p), ("z_stride", C.c_int64), ("x_stride", C.c_int64), ("g_stride", C.c_int64),
                 ("z_bias", C.c_void_p), ("x_bias", C.c_void_p), ("seq_info", C.c_void_p), ("n_seq", C.c_int32), ("state", C.c_void_p), ("slot_stride", C.c_int64),
                 ("dst", C.c_void_p), ("dst_stride", C.c_int64), ("width", C.c_int32), ("n_tokens", C.c_int32)]
+
+
+class NormChainArgs(C.Structure):
+    """b200_norm_chain_args (include/b200_ggml_ops.h); strides in floats."""
+    _fields_ = [("y", C.c_void_p), ("y_s_slot", C.c_int64), ("y_s_tok", C.c_int64), ("yw", C.c_void_p), ("yw_s_tok", C.c_int64), ("shared", C.c_void_p), ("shared_stride", C.c_int64),
+                ("res", C.c_void_p), ("res_stride", C.c_int64), ("w1", C.c_void_p), ("b1", C.c_void_p), ("w2", C.c_void_p), ("b2", C.c_void_p), ("x", C.c_void_p),
+                ("x_stride", C.c_int64), ("h", C.c_void_p), ("h_stride", C.c_int64), ("n", C.c_int64), ("n_tok", C.c_int64), ("n_y", C.c_int32), ("kind1", C.c_int32),
+                ("kind2", C.c_int32), ("y_scale", C.c_float), ("eps", C.c_float)]
+
+
+class TokenShiftArgs(C.Structure):
+    """b200_token_shift_args (include/b200_ggml_ops.h); strides in floats."""
+    _fields_ = [("h", C.c_void_p), ("h_stride", C.c_int64), ("mu", C.c_void_p), ("seq_info", C.c_void_p), ("n_seq", C.c_int32), ("prev", C.c_void_p), ("slot_stride", C.c_int64),
+                ("dst", C.c_void_p), ("dst_s_mix", C.c_int64), ("dst_s_tok", C.c_int64), ("width", C.c_int32), ("n_mix", C.c_int32), ("n_tokens", C.c_int32)]
+
+
+class TimeMixArgs(C.Structure):
+    """b200_time_mix_args (include/b200_ggml_ops.h); strides in floats."""
+    _fields_ = [("r", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("z", C.c_void_p), ("r_stride", C.c_int64), ("k_stride", C.c_int64), ("v_stride", C.c_int64),
+                ("z_stride", C.c_int64), ("w0", C.c_void_p), ("u", C.c_void_p), ("seq_info", C.c_void_p), ("n_seq", C.c_int32), ("state", C.c_void_p), ("slot_stride", C.c_int64),
+                ("dst", C.c_void_p), ("dst_stride", C.c_int64), ("heads", C.c_int32), ("dim", C.c_int32)]
 
 
 _SIGS = {
@@ -227,6 +250,9 @@ _OPS_SIGS = {
     "b200_op_short_conv": (C.c_int, [C.POINTER(ShortConvArgs), C.c_void_p]),
     "b200_op_delta_rule_scan": (C.c_int, [C.POINTER(DeltaRuleArgs), C.c_void_p]),
     "b200_op_mingru_scan": (C.c_int, [C.POINTER(MinGruArgs), C.c_void_p]),
+    "b200_op_norm_chain": (C.c_int, [C.POINTER(NormChainArgs), C.c_void_p]),
+    "b200_op_token_shift": (C.c_int, [C.POINTER(TokenShiftArgs), C.c_void_p]),
+    "b200_op_time_mix_scan": (C.c_int, [C.POINTER(TimeMixArgs), C.c_void_p]),
 }
 
 _lib = None

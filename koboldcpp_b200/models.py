@@ -4,7 +4,7 @@ from __future__ import annotations
 import json
 from pathlib import Path
 
-from . import galirax, genesun, medodra, zevopel
+from . import galirax, genesun, mafuzen, medodra, zevopel
 from .lib import B200Error
 
 ARCHITECTURES = {
@@ -12,6 +12,7 @@ ARCHITECTURES = {
     "Galirax": galirax.load,
     "Zevopel": zevopel.load,
     "Medodra": medodra.load,
+    "Mafuzen": mafuzen.load,
 }
 
 
