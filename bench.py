@@ -910,6 +910,121 @@ def medodra_beside_config(size: str) -> dict:
     return {"architecture": "Galirax", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": [att if il % 2 == 0 else lin for il in range(DESIGN_LAYERS)]}
 
 
+# ------------------------------------------------------------------------------------------------ --design mafuzen
+# The same measurement for the Mafuzen design (attention with a distance penalty, retention, windowed attention beside time mixing, and
+# attention over the first layer's cache in turn; table-routed experts plus a shared one and a per-layer token input in every layer),
+# beside the closest existing model of the framework: Galirax with attention, lightning (linear attention), windowed attention and
+# attention layers in turn and routed experts in every layer at equal width, depth, heads and expert size.
+MAFUZEN_SIDE, MAFUZEN_RANK = 256, 64
+
+
+def mafuzen_config(size: str) -> dict:
+    import math
+    W, (h, g, d, v), (ne, top, ff, _ng, _nk), window = GALIRAX_SIZES[size]
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": ne, "top": top}, "shared": {"ff": ff}}
+    layers = []
+    for il in range(DESIGN_LAYERS):
+        att = {"heads": h, "kv_heads": g, "dim": d, "vdim": v, "scale": 1.0 / math.sqrt(d)}
+        if il % 4 == 1:
+            mixer = {"heads": h, "dim": d, "vdim": v, "rot": {"base": 10000.0, "dims": d}, "decay": [1.0 - 2.0 ** (-5 - 3 * i / h) for i in range(h)]}
+        elif il % 4 == 2:
+            mixer = {"left": dict(att, mask={"size": window, "keep_first": 4}), "left_scale": 0.7, "right": {"heads": W // 64, "dim": 64}, "right_scale": 0.8}
+        else:
+            mixer = att if il % 4 == 0 else dict(att, kv_from=il - 3)
+        layers.append({"type": ("attention", "retention", "parallel", "attention")[il % 4], "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Mafuzen", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "token_side": {"dim": MAFUZEN_SIDE}, "layers": layers}
+
+
+def mafuzen_random_tensors(cfg: dict):
+    W, V = cfg["width"], cfg["vocab"]
+    ES = cfg["token_side"]["dim"]
+    t = {"embed": (V, W), "final.norm": (W,), "final.norm.b": (W,), "side.embed": (V, ES * len(cfg["layers"]))}
+    for i, L in enumerate(cfg["layers"]):
+        p, mx = f"l{i}.", L["mixer"]
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            t.update({p + n: (W,), p + n + ".b": (W,)})
+        t.update({p + "side.gate": (ES, W), p + "side.proj": (W, ES), p + "side.norm": (W,)})
+        if L["type"] == "retention":
+            H, D, Vd = mx["heads"], mx["dim"], mx["vdim"]
+            t.update({p + "mix.q": (H * D, W), p + "mix.k": (H * D, W), p + "mix.v": (H * Vd, W), p + "mix.g": (H * Vd, W), p + "mix.o": (W, H * Vd)})
+        elif L["type"] == "attention":
+            H, G, D, Vd = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
+            t.update({p + "mix.q": (H * D, W), p + "mix.o": (W, H * Vd)})
+            if "kv_from" not in mx:
+                t.update({p + "mix.k": (G * D, W), p + "mix.v": (G * Vd, W)})
+        else:
+            a, HD = mx["left"], mx["right"]["heads"] * mx["right"]["dim"]
+            H, G, D = a["heads"], a["kv_heads"], a["dim"]
+            t.update({p + "mix.left.q": (H * D, W), p + "mix.left.k": (G * D, W), p + "mix.left.g": (H * D, W), p + "mix.left.o": (W, H * D)})
+            t.update({p + "mix.right.mu." + x: (W,) for x in "rkvgw"})
+            t.update({p + "mix.right." + x: (HD, W) for x in "rkvg"})
+            t.update({p + "mix.right.w1": (MAFUZEN_RANK, W), p + "mix.right.w2": (HD, MAFUZEN_RANK), p + "mix.right.w0": (HD,), p + "mix.right.u": (mx["right"]["heads"], mx["right"]["dim"]),
+                      p + "mix.right.norm": (HD,), p + "mix.right.o": (W, HD)})
+        E, top, F, FS = L["mlp"]["router"]["experts"], L["mlp"]["router"]["top"], L["mlp"]["expert"]["ff"], L["mlp"]["shared"]["ff"]
+        t.update({p + "mlp.shared.up": (FS, W), p + "mlp.shared.down": (W, FS), p + "mlp.table": (V, top)})
+        for e in range(E):
+            t.update({f"{p}mlp.e{e}.up": (F, W), f"{p}mlp.e{e}.down": (W, F)})
+    out = random_tensors({k: x for k, x in t.items() if not k.endswith(".table")})
+    rng = np.random.default_rng(4)
+    for name, shape in t.items():
+        if name.endswith(".table"):  # the chosen experts of a token differ: a random start, then neighbours
+            E = cfg["layers"][int(name[1:name.index(".")])]["mlp"]["router"]["experts"]
+            ids = (rng.integers(0, E, (shape[0], 1)) + np.arange(shape[1])) % E
+            out[name] = ("I32", shape, ids.astype(np.int32).reshape(-1).view(np.uint8))
+        elif name.endswith(".right.w0"):  # decays exp(-exp(w0)) between 0.5 and 0.999
+            out[name] = ("F32", shape, np.linspace(-7.0, -0.4, shape[0], dtype=np.float32).view(np.uint8))
+        elif ".mu." in name:
+            out[name] = ("F32", shape, np.full(shape[0], 0.5, np.float32).view(np.uint8))
+        elif name.endswith(".b"):
+            out[name] = ("F32", shape, np.zeros(shape[0], np.float32).view(np.uint8))
+    return out
+
+
+def mafuzen_step_cost(cfg: dict, n_tokens: int, n_seq: int, ctx: int) -> dict:
+    """Algorithmic bytes (bf16 weights once -- of the experts those a batch of this size can reach --, the visible f32 cache rows and the
+    recurrent states of the batch) and FLOPs of one step."""
+    W, V, ES = cfg["width"], cfg["vocab"], cfg["token_side"]["dim"]
+    wparams = active = W * V
+    cache = state = attn_flop = 0
+    for L in cfg["layers"]:
+        mx = L["mixer"]
+        if L["type"] == "retention":
+            H, D, Vd = mx["heads"], mx["dim"], mx["vdim"]
+            p = W * (2 * H * D + 2 * H * Vd) + W * H * Vd
+            state += n_seq * H * D * Vd * 4 * 2
+            attn_flop += 4 * n_tokens * H * D * Vd
+        else:
+            par = L["type"] == "parallel"
+            a = mx["left"] if par else mx
+            H, G, D, Vd = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            p = W * H * D + W * H * Vd + (0 if "kv_from" in a else W * G * D + (0 if par else W * G * Vd))
+            win = (a.get("mask") or {}).get("size", 0)
+            vis = min(ctx, win) if win else ctx
+            cache += n_seq * vis * G * (D + Vd) * 4
+            attn_flop += 2 * n_tokens * H * (vis if n_tokens == n_seq or win else ctx // 2) * (D + Vd)
+            if par:
+                HR, DR = mx["right"]["heads"], mx["right"]["dim"]
+                p += W * H * Vd + 5 * W * HR * DR + MAFUZEN_RANK * (W + HR * DR)  # the gate; r, k, v, g, o; the decay
+                state += n_seq * HR * DR * DR * 4 * 2
+                attn_flop += 4 * n_tokens * HR * DR * DR
+        r, F, FS = L["mlp"]["router"], L["mlp"]["expert"]["ff"], L["mlp"]["shared"]["ff"]
+        wparams += p + 2 * W * F * min(r["experts"], n_tokens * r["top"]) + 2 * W * FS + 2 * W * ES
+        active += p + 2 * W * F * r["top"] + 2 * W * FS + 2 * W * ES
+    return {"weight_bytes": 2 * wparams, "cache_bytes": cache, "state_bytes": state, "flop": 2 * active * n_tokens + attn_flop}
+
+
+def mafuzen_beside_config(size: str) -> dict:
+    """Galirax at equal width, depth, heads and expert size: attention, lightning, windowed attention and attention layers in turn."""
+    import math
+    W, (h, g, d, v), (ne, top, ff, ng, nk), window = GALIRAX_SIZES[size]
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": ne, "top": top, "groups": {"count": ng, "keep": nk}, "scale": 2.0}}
+    rot = {"base": 500000.0, "dims": d // 2}
+    att = {"type": "attention", "mixer": {"heads": h, "kv_heads": g, "dim": d, "vdim": v, "rot": rot, "scale": 1.0 / math.sqrt(d)}, "mlp": mlp}
+    lin = {"type": "lightning", "mixer": {"heads": h, "dim": d, "vdim": v, "decay": [1.0 - 2.0 ** (-5 - 3 * i / h) for i in range(h)]}, "mlp": mlp}
+    win = {"type": "attention_2", "mixer": dict(att["mixer"], mask={"size": window, "keep_first": 4}), "mlp": mlp}
+    return {"architecture": "Galirax", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": [(att, lin, win, att)[il % 4] for il in range(DESIGN_LAYERS)]}
+
+
 def galirax_llama_shape(size: str):
     import koboldcpp_b200.llama as LL
     W, (h, g, d, v), (ne, top, ff, ng, nk), window = GALIRAX_SIZES[size]
@@ -947,8 +1062,12 @@ def random_tensors(shapes: dict, seed: int = 1):
 
 
 def design_table():
-    from koboldcpp_b200 import galirax, genesun, medodra, zevopel
+    from koboldcpp_b200 import galirax, genesun, mafuzen, medodra, zevopel
     return {
+        "mafuzen": {"sizes": GALIRAX_SIZES, "config": mafuzen_config, "tensors": mafuzen_random_tensors, "cost": mafuzen_step_cost, "build": mafuzen.build,
+                    "beside_design": {"name": "galirax", "config": mafuzen_beside_config, "tensors": lambda cfg: random_tensors(galirax_tensor_shapes(cfg)),
+                                      "cost": galirax_step_cost, "build": galirax.build},
+                    "beside": "Galirax (attention, lightning, windowed attention and attention layers in turn, routed experts in every layer), equal width / depth / heads / expert size, bf16"},
         "medodra": {"sizes": GALIRAX_SIZES, "config": medodra_config, "tensors": medodra_random_tensors, "cost": medodra_step_cost, "build": medodra.build,
                     "beside_design": {"name": "galirax", "config": medodra_beside_config, "tensors": lambda cfg: random_tensors(galirax_tensor_shapes(cfg)),
                                       "cost": galirax_step_cost, "build": galirax.build},
@@ -1021,7 +1140,7 @@ def design_leg(args) -> int:
             t0 = time.time()
             n_e2e = 8
             for _ in range(n_e2e):
-                lg = eng.step([(rid, [5], [0]) for rid in ids])
+                lg = eng.step([(rid, [5 + i], [0]) for i, rid in enumerate(ids)])
             e2e_ms = (time.time() - t0) / n_e2e * 1e3
             ms = time_replay(m, m.stream, steps, warmup)
             cost = DS["cost"](cfg, nseq, nseq, DESIGN_CTX)
@@ -1084,7 +1203,7 @@ def main() -> int:
     ap.add_argument("--cpu-budget", type=float, default=18.0)
     ap.add_argument("--no-tp70", action="store_true", default=bool(os.environ.get("B200_BENCH_NO_TP70")),
                     help="skip the auxiliary 70B tensor-parallel leg (BASELINE.json configs[4])")
-    ap.add_argument("--design", default="", choices=["", "genesun", "galirax", "zevopel", "medodra"],
+    ap.add_argument("--design", default="", choices=["", "genesun", "galirax", "zevopel", "medodra", "mafuzen"],
                     help="instead of the default workload: prefill / decode of this design at real layer shapes beside the closest existing model at equal size")
     ap.add_argument("--design-sizes", default="", help="comma-separated subset of the sizes of the design (genesun: " + ",".join(DESIGN_SIZES) + "; the others: " + ",".join(GALIRAX_SIZES) + ")")
     args = ap.parse_args()

@@ -202,6 +202,9 @@ B200_API int b200_mul_mat_id_q(int type, const void *as, size_t w_row_bytes, siz
  * The call first converts X to bf16 at the front of the workspace.  X == NULL: the workspace still holds the converted activations
  * of the previous call with the same K and N (sibling matmuls over one activation: Q / K / V, gate / up) and they are used as is. */
 B200_API size_t b200_mul_mat_q_workspace_bytes(int type, int64_t K, int64_t M, int64_t N);
+/* 0, or 1 once a dense bf16 GEMM of this process has given up waiting for its own pipeline (its results are then not stored); meaningful
+ * after a synchronisation of the stream. */
+B200_API int b200_gemm_status(void);
 B200_API int b200_mul_mat_q(int type, const void *W, size_t w_row_bytes, const float *X, int64_t x_stride,
                             float *dst, int64_t dst_stride, int64_t K, int64_t M, int64_t N,
                             void *workspace, size_t workspace_bytes, b200_stream_t stream);

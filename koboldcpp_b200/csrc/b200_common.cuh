@@ -141,6 +141,26 @@ __device__ __forceinline__ void mbar_wait(unsigned long long *bar, unsigned pari
         "r"(parity)
         : "memory");
 }
+// The same with a limit: false when the phase has not completed within `limit` clock cycles (nothing is consumed then).
+__device__ __forceinline__ bool mbar_wait_limited(unsigned long long *bar, unsigned parity, long long limit) {
+    long long t0 = 0;
+    for (unsigned i = 0;; i++) {
+        unsigned done;
+        asm volatile(
+            "{\n"
+            ".reg .pred p;\n"
+            "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+            "selp.u32 %0, 1, 0, p;\n"
+            "}\n"
+            : "=r"(done)
+            : "r"(smem_u32(bar)), "r"(parity)
+            : "memory");
+        if (done) return true;
+        const long long now = clock64();
+        if (i == 0) t0 = now;
+        else if (now - t0 > limit) return false;
+    }
+}
 // global -> shared bulk copy; dst/src 16-byte aligned, bytes % 16 == 0; completes on `bar` (complete_tx)
 __device__ __forceinline__ void bulk_g2s(void *dst, const void *src, unsigned bytes, unsigned long long *bar) {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),

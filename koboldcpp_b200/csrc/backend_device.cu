@@ -203,6 +203,7 @@ ggml_backend_t ggml_backend_b200_init(int device) {
         return nullptr;
     }
     B200_CHECK_CUDA(cudaSetDevice(device));
+    if (!g_dry) b200::gemm_status_prepare();
     BackendCtx *c = new BackendCtx{device, "B200_" + std::to_string(device), graph_exec_new(device)};
     return new ggml_backend{&k_guid, k_backend_iface, device_get(device), c};
 }

@@ -20,6 +20,9 @@
 // launch count) and zero-fills the outputs instead of launching.  It exists so that the reference's own llama.cpp +
 // ggml_backend_sched can drive the vtables in CI; NOTHING is computed (this is not a CPU fallback: results are zeros).
 namespace b200 {
+// mmq.cu: the host word that a dense GEMM whose pipeline gave up sets (b200_gemm_status)
+void gemm_status_prepare();
+
 extern bool g_dry;
 extern int g_dry_devices;
 namespace dry {

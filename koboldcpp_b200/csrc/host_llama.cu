@@ -317,6 +317,7 @@ extern "C" int b200_llama_decode_batch(b200_llama *m, const int32_t *tokens, con
     LL_REQUIRE(st == GGML_STATUS_SUCCESS, B200_ERR_CUDA, "b200_llama_decode_batch: graph_compute failed (%d)", (int)st);
     if (n_out > 0) be->iface.get_tensor_async(be, m->logits_t, logits, 0, 4 * (size_t)hp.n_vocab * (size_t)n_out);
     be->iface.synchronize(be);
+    LL_REQUIRE(b200_gemm_status() == 0, B200_ERR_CUDA, "b200_llama_decode_batch: a product gave up waiting for its operands: the step's results are invalid");
     return B200_OK;
 }
 

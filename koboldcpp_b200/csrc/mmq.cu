@@ -403,6 +403,7 @@ struct MmqParams {
     int n_batch;
     size_t w_batch_bytes;
     int64_t dst_batch, n_pad;
+    int n_expert;  // grouped: experts in the stack
 };
 
 template <int TYPE, int BN>
@@ -875,7 +876,130 @@ __global__ void __launch_bounds__(MQ2_THREADS, 1) mmq_tc2_kernel(const __grid_co
     }
 }
 
+// ================================================================ dense bf16 weights: both operands by TMA
+// Dense rows need no unpacking, so nothing stands between HBM and the tensor core: one warp's elected lane requests the weight tile
+// [128 rows x 64] and the activation tile [BN rows x 64] of every stage (128-byte swizzle by the copy engine) as soon as the stage is
+// free, one lane issues the MMAs, four warps read the accumulators out of TMEM.  The stages are as many as shared memory takes, all
+// of them in flight.  Every wait has a limit: a role that gives up says so in shared memory, the others run into their own limits, the
+// copies in flight are waited for, TMEM is freed, nothing is stored and *timeout is set.
+constexpr long long BG_WAIT_LIMIT = 4000000000LL;  // clock cycles: about two seconds
+template <int BN> constexpr int bg_stages() { return BN >= 256 ? 4 : BN >= 128 ? 6 : 8; }
+template <int BN, bool GROUPED>
+__global__ void __launch_bounds__(MQ2_THREADS, 1) bf16_gemm_kernel(const __grid_constant__ TmapBytes tmA, const __grid_constant__ TmapBytes tmB, const __grid_constant__ MmqParams p,
+                                                                   int64_t w_rows_per_product, int *timeout) {
+    constexpr int STAGES = bg_stages<BN>(), A_BYTES = MQ_BM * MQ_BK * 2, B_BYTES = BN * MQ_BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
+    int64_t n0 = (int64_t)blockIdx.y * BN, n_end = p.N, a_row = (int64_t)blockIdx.x * MQ_BM;
+    const int64_t m0 = a_row;
+    if constexpr (GROUPED) {  // uniform over the CTA: tiles past the table's end have nothing to do
+        if ((int)blockIdx.y >= __ldg(p.tile_tab)) return;
+        const int *te = p.tile_tab + 1 + 3 * blockIdx.y;
+        a_row += (int64_t)__ldg(te) * w_rows_per_product;
+        n0 = __ldg(te + 1);
+        n_end = __ldg(te + 2);
+    }
+    extern __shared__ unsigned char smem_raw[];
+    unsigned char *smem = reinterpret_cast<unsigned char *>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+    __shared__ __align__(8) unsigned long long full_bar[STAGES], empty_bar[STAGES], tmem_full_bar;
+    __shared__ unsigned tmem_base_s;
+    __shared__ volatile int failed;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
+    const int nkb_all = (int)(p.K / MQ_BK);
+    const int ksplit = GROUPED ? 1 : p.ksplit;  // split-K: this CTA's steps [kb0, kb0 + nkb)
+    const bool batched = !GROUPED && p.n_batch > 1;
+    const int zk = batched ? 0 : (int)blockIdx.z, zb = batched ? (int)blockIdx.z : 0;
+    a_row += zb * w_rows_per_product;
+    const int kb0 = (int)(((int64_t)zk * nkb_all) / ksplit), nkb = (int)(((int64_t)(zk + 1) * nkb_all) / ksplit) - kb0;
+
+    if (tid == 0) {
+        for (int s = 0; s < STAGES; s++) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
+        mbar_init(&tmem_full_bar, 1);
+        failed = 0;
+        mbar_fence_init();
+    }
+    if (warp == 4) tmem_alloc(&tmem_base_s, BN);
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const unsigned tmem_base = tmem_base_s;
+
+    if (warp == 5) {
+        if (lane == 0) {
+            int kb = 0;
+            for (; kb < nkb; kb++) {
+                const int s = kb % STAGES;
+                if (!mbar_wait_limited(&empty_bar[s], ((unsigned)(kb / STAGES) & 1u) ^ 1u, BG_WAIT_LIMIT)) { failed = 1; break; }
+                unsigned char *st = smem + (size_t)s * STAGE_BYTES;
+                mbar_expect_tx(&full_bar[s], (unsigned)STAGE_BYTES);
+                tma_load_2d(st, &tmA, (kb0 + kb) * MQ_BK, (int)a_row, &full_bar[s]);
+                tma_load_2d(st + A_BYTES, &tmB, (kb0 + kb) * MQ_BK, (int)n0 + (batched ? zb * (int)p.n_pad : 0), &full_bar[s]);
+            }
+            if (kb < nkb)  // gave up: the copies that were requested still have to land before this CTA may end
+                for (int j = kb > STAGES ? kb - STAGES : 0; j < kb; j++) mbar_wait_limited(&full_bar[j % STAGES], (unsigned)(j / STAGES) & 1u, BG_WAIT_LIMIT);
+        }
+    } else if (warp == 4) {
+        constexpr unsigned idesc = umma_idesc_bf16(MQ_BM, BN);
+        int kb = 0;
+        for (; kb < nkb; kb++) {
+            const int s = kb % STAGES;
+            const bool ok = mbar_wait_limited(&full_bar[s], (unsigned)(kb / STAGES) & 1u, BG_WAIT_LIMIT);
+            if (!__all_sync(0xffffffffu, ok)) { failed = 1; break; }
+            tc_fence_after();
+            if (lane == 0) {
+                const unsigned a_addr = smem_u32(smem + (size_t)s * STAGE_BYTES), b_addr = a_addr + A_BYTES;
+#pragma unroll
+                for (int k = 0; k < MQ_BK / 16; k++)
+                    tc_mma_bf16(tmem_base, umma_desc_sw128(a_addr) + 2u * k, umma_desc_sw128(b_addr) + 2u * k, idesc, (kb | k) != 0 ? 1u : 0u);
+                tc_commit(&empty_bar[s]);
+                if (kb == nkb - 1) tc_commit(&tmem_full_bar);
+            }
+            __syncwarp();
+        }
+        if (kb < nkb && lane == 0) tc_commit(&tmem_full_bar);  // gave up: releases the epilogue once the MMAs issued so far have retired
+        __syncwarp();
+        tc_fence_before();
+    } else {
+        bool ok = mbar_wait_limited(&tmem_full_bar, 0u, 3 * BG_WAIT_LIMIT);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) failed = 1;
+        tc_fence_after();
+        const int64_t m = m0 + tid;
+        const bool row_ok = m < p.M && ok && !failed;
+        float *drow = p.dst + m + (batched ? (int64_t)zb * p.dst_batch : 0);
+#pragma unroll 1
+        for (int c0 = 0; c0 < BN; c0 += 32) {
+            float v[32];
+            tmem_ld32(tmem_base + ((unsigned)(warp * 32) << 16) + (unsigned)c0, v);
+            if (row_ok) {
+#pragma unroll
+                for (int j = 0; j < 32; j++) {
+                    const int64_t n = n0 + c0 + j;
+                    if (n >= n_end) continue;
+                    if constexpr (GROUPED) drow[(int64_t)__ldg(p.row_dst + n)] = v[j];  // scatter: sorted row -> (token, slot)
+                    else if (ksplit > 1) atomicAdd(drow + n * p.dst_stride, v[j]);      // (result unused: RED.ADD.F32)
+                    else drow[n * p.dst_stride] = v[j];
+                }
+            }
+        }
+        tc_fence_before();
+    }
+    __syncthreads();
+    if (tid == 0 && failed && timeout) atomicExch(timeout, 1);
+    if (warp == 4) {
+        tc_fence_after();
+        tmem_dealloc(tmem_base, BN);
+    }
+}
+
 // ---------------------------------------------------------------- host side
+// set by a GEMM whose pipeline gave up; pinned host memory, so that reading it after a synchronisation costs nothing
+static int *g_gemm_timeout = nullptr;
+void gemm_status_prepare() {
+    if (g_gemm_timeout) return;
+    int *p = nullptr;
+    if (cudaHostAlloc((void **)&p, sizeof(int), cudaHostAllocPortable | cudaHostAllocMapped) == cudaSuccess) { *p = 0; g_gemm_timeout = p; }
+    else cudaGetLastError();
+}
+
 static int64_t mmq_bn(int64_t N) { return N <= 32 ? 32 : N <= 64 ? 64 : N <= 128 ? 128 : 256; }
 static int64_t mmq_n_pad(int64_t N) { const int64_t bn = mmq_bn(N); return (N + bn - 1) / bn * bn; }
 
@@ -908,8 +1032,59 @@ static EncodeTiledFn encode_tiled_fn() {
     return fn;
 }
 
+// a 2-D bf16 tensor map of `rows` rows of K values, boxes of `box_rows` x 64, 128-byte swizzle
+static int encode_rows(TmapBytes &tm, const void *base, int64_t K, int64_t rows, size_t row_bytes, int box_rows) {
+    EncodeTiledFn enc = encode_tiled_fn();
+    if (!enc) { set_error("b200_mul_mat_q: cuTensorMapEncodeTiled not available"); return B200_ERR_CUDA; }
+    const unsigned long long gdim[2] = {(unsigned long long)K, (unsigned long long)rows}, gstr[1] = {(unsigned long long)row_bytes};
+    const unsigned box[2] = {(unsigned)MQ_BK, (unsigned)box_rows}, estr[2] = {1, 1};
+    // CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 = 9, INTERLEAVE_NONE = 0, SWIZZLE_128B = 3, L2_PROMOTION_L2_256B = 3, FLOAT_OOB_FILL_NONE = 0
+    const int rc = enc(&tm, 9, 2, (void *)base, gdim, gstr, box, estr, 0, 3, 3, 0);
+    if (rc != 0) { set_error("b200_mul_mat_q: cuTensorMapEncodeTiled failed (%d)", rc); return B200_ERR_CUDA; }
+    return B200_OK;
+}
+
+template <int BN, bool GROUPED>
+static int bf16_gemm_launch(const MmqParams &p, int64_t n_pad, int64_t w_rows_per_product, cudaStream_t st, unsigned grid_y) {
+    constexpr size_t smem = (size_t)bg_stages<BN>() * (MQ_BM * MQ_BK * 2 + BN * MQ_BK * 2) + 1024;
+    static bool attr_set_dev[16] = {};  // cudaFuncSetAttribute is per device
+    int cur_dev = 0;
+    B200_CUDA_TRY(cudaGetDevice(&cur_dev));
+    bool &attr_set = attr_set_dev[cur_dev & 15];
+    if (!attr_set) {
+        B200_CUDA_TRY(cudaFuncSetAttribute(bf16_gemm_kernel<BN, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        attr_set = true;
+    }
+    const int64_t products = GROUPED ? p.n_expert : p.n_batch;
+    TmapBytes tmA, tmB;
+    int rc = encode_rows(tmA, p.W, p.K, (products - 1) * w_rows_per_product + p.M, p.w_row_bytes, MQ_BM);
+    if (rc != B200_OK) return rc;
+    rc = encode_rows(tmB, p.Xb, p.K, n_pad * (p.n_batch > 1 ? p.n_batch : 1), (size_t)p.K * 2, BN);
+    if (rc != B200_OK) return rc;
+    dim3 grid((unsigned)((p.M + MQ_BM - 1) / MQ_BM), GROUPED ? grid_y : (unsigned)((p.N + BN - 1) / BN));
+    MmqParams q = p;
+    q.ksplit = 1;
+    if (p.n_batch > 1) {
+        grid.z = (unsigned)p.n_batch;
+    } else if (!GROUPED && (int64_t)grid.x * grid.y * 2 <= 148 && p.K >= 2048) {
+        // fewer tiles than half the SMs: two CTAs share a tile's K range and add into a zeroed dst (two partials only: the sum is
+        // independent of the arrival order)
+        q.ksplit = 2;
+        grid.z = 2;
+        if (p.dst_stride == p.M) B200_CUDA_TRY(cudaMemsetAsync(p.dst, 0, (size_t)p.M * p.N * sizeof(float), st));
+        else B200_CUDA_TRY(cudaMemset2DAsync(p.dst, (size_t)p.dst_stride * sizeof(float), 0, (size_t)p.M * sizeof(float), (size_t)p.N, st));
+    }
+    bf16_gemm_kernel<BN, GROUPED><<<grid, MQ2_THREADS, smem, st>>>(tmA, tmB, q, w_rows_per_product, g_gemm_timeout);
+    B200_CUDA_TRY(cudaGetLastError());
+    return B200_OK;
+}
+
 template <int TYPE, int BN, bool GROUPED = false>
 static int mmq2_launch(const MmqParams &p, int64_t n_pad, cudaStream_t st, unsigned grid_y = 0) {
+    if constexpr (TYPE == B200_TYPE_BF16) {  // products whose weight rows lie at one stride over all of them: one tensor map covers the stack
+        const size_t step = GROUPED ? p.expert_bytes : p.n_batch > 1 ? p.w_batch_bytes : 0;
+        if (step % p.w_row_bytes == 0) return bf16_gemm_launch<BN, GROUPED>(p, n_pad, (int64_t)(step / p.w_row_bytes), st, grid_y);
+    }
     constexpr size_t smem = (size_t)MQ2_STAGES * (MQ_BM * MQ_BK * 2 + BN * MQ_BK * 2) + 1024;
     static bool attr_set_dev[16] = {};  // cudaFuncSetAttribute is per device
     int cur_dev = 0;
@@ -954,7 +1129,10 @@ template <int TYPE>
 static int mmq_dispatch_bn(const MmqParams &p, cudaStream_t st) {
     if constexpr (TYPE == B200_TYPE_BF16) {  // dense rows: the asynchronous kernel only, any K that is a multiple of the K step
         const int64_t n_pad = mmq_n_pad(p.N);
-        switch (mmq_bn(p.N)) {
+        // few rows of weights: narrower tiles until they fill the device at least by half (with the two halves of K)
+        int64_t bn = mmq_bn(p.N);
+        while (bn > 32 && (p.M + MQ_BM - 1) / MQ_BM * ((p.N + bn - 1) / bn) * p.n_batch * 4 <= 148) bn /= 2;
+        switch (bn) {
             case 32: return mmq2_launch<TYPE, 32>(p, n_pad, st);
             case 64: return mmq2_launch<TYPE, 64>(p, n_pad, st);
             case 128: return mmq2_launch<TYPE, 128>(p, n_pad, st);
@@ -1064,6 +1242,8 @@ static int mid_dispatch_bn(const MmqParams &p, int64_t bn, int64_t n_rows, unsig
 
 using namespace b200;
 
+extern "C" int b200_gemm_status(void) { return g_gemm_timeout ? *(volatile int *)g_gemm_timeout : 0; }
+
 extern "C" size_t b200_mul_mat_q_workspace_bytes(int type, int64_t K, int64_t M, int64_t N) {
     (void)type; (void)M;
     if (K <= 0 || N <= 0) return 0;
@@ -1107,7 +1287,7 @@ extern "C" int b200_mul_mat_q(int type, const void *W, size_t w_row_bytes, const
     MmqParams p;
     p.W = (const unsigned char *)W; p.w_row_bytes = w_row_bytes; p.Xb = xb; p.dst = dst; p.dst_stride = dst_stride; p.K = K; p.M = M; p.N = N;
     p.tile_tab = nullptr; p.row_dst = nullptr; p.expert_bytes = 0;
-    p.n_batch = 1; p.w_batch_bytes = 0; p.dst_batch = 0; p.n_pad = n_pad;
+    p.n_batch = 1; p.w_batch_bytes = 0; p.dst_batch = 0; p.n_pad = n_pad; p.n_expert = 1;
     switch (type) {
         case B200_TYPE_Q4_0: return mmq_dispatch_bn<B200_TYPE_Q4_0>(p, st);
         case B200_TYPE_Q8_0: return mmq_dispatch_bn<B200_TYPE_Q8_0>(p, st);
@@ -1148,7 +1328,7 @@ extern "C" int b200_mul_mat_bf16_batched(const void *W, size_t w_row_bytes, size
     MmqParams p;
     p.W = (const unsigned char *)W; p.w_row_bytes = w_row_bytes; p.Xb = xb; p.dst = dst; p.dst_stride = dst_stride; p.K = K; p.M = M; p.N = N;
     p.tile_tab = nullptr; p.row_dst = nullptr; p.expert_bytes = 0;
-    p.n_batch = n_batch; p.w_batch_bytes = w_batch_bytes; p.dst_batch = dst_batch; p.n_pad = n_pad;
+    p.n_batch = n_batch; p.w_batch_bytes = w_batch_bytes; p.dst_batch = dst_batch; p.n_pad = n_pad; p.n_expert = 1;
     return mmq_dispatch_bn<B200_TYPE_BF16>(p, st);
 }
 
@@ -1209,7 +1389,7 @@ extern "C" int b200_mul_mat_id_q(int type, const void *as, size_t w_row_bytes, s
     MmqParams p;
     p.W = (const unsigned char *)as; p.w_row_bytes = w_row_bytes; p.Xb = xb; p.dst = dst; p.dst_stride = 0; p.K = K; p.M = M; p.N = n_rows;
     p.tile_tab = t.tile_tab; p.row_dst = t.row_dst; p.expert_bytes = expert_bytes;
-    p.n_batch = 1; p.w_batch_bytes = 0; p.dst_batch = 0; p.n_pad = 0;
+    p.n_batch = 1; p.w_batch_bytes = 0; p.dst_batch = 0; p.n_pad = 0; p.n_expert = n_expert;
     switch (type) {
         case B200_TYPE_Q4_0: return mid_dispatch_bn<B200_TYPE_Q4_0>(p, bn, n_rows, (unsigned)max_tiles, st);
         case B200_TYPE_Q8_0: return mid_dispatch_bn<B200_TYPE_Q8_0>(p, bn, n_rows, (unsigned)max_tiles, st);

@@ -184,6 +184,13 @@ __global__ void unary_kernel(int op, const float *__restrict__ x, float *__restr
     if (i < n) dst[i] = unary_apply(op, x[i], p0, p1);
 }
 
+__global__ void unary4_kernel(int op, const float4 *__restrict__ x, float4 *__restrict__ dst, int64_t n4, float p0, float p1) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n4) return;
+    const float4 v = x[i];
+    dst[i] = make_float4(unary_apply(op, v.x, p0, p1), unary_apply(op, v.y, p0, p1), unary_apply(op, v.z, p0, p1), unary_apply(op, v.w, p0, p1));
+}
+
 // ------------------------------------------------------------------------------------------------ ROPE
 // T = float, or __half for the in-place K-shift over an f16 cache (build_k_shift, src/llama.cpp:10144-10192; reference rope.cu f16 path)
 template <typename T> struct RopeIO;
@@ -466,6 +473,20 @@ __global__ void get_rows_kernel(TD src, int type, TD ids, TD dst) {
     const bool ok = r >= 0 && r < src.ne[1];
     const unsigned char *row = (const unsigned char *)(src.data + (int64_t)(ok ? r : 0) * src.nb[1] + i11 * src.nb[2] + i12 * src.nb[3]);
     for (int64_t c = threadIdx.x; c < dst.ne[0]; c += blockDim.x) out[c] = ok ? dq_value(type, row, c) : __int_as_float(0x7fc00000);
+}
+
+// f32 rows (or any 32-bit words): a CTA per 1024 values of a row
+__global__ void __launch_bounds__(256) get_rows_f32_kernel(TD src, TD ids, TD dst, bool vec4) {
+    const int64_t c0 = (int64_t)blockIdx.x * 1024 + threadIdx.x * 4, i10 = blockIdx.y;
+    const int32_t r = *(const int32_t *)(ids.data + i10 * ids.nb[0]);
+    const bool ok = r >= 0 && r < src.ne[1];
+    const float *row = (const float *)(src.data + (int64_t)(ok ? r : 0) * src.nb[1]);
+    float *out = (float *)(dst.data + i10 * dst.nb[1]);
+    if (vec4 && ok) {
+        if (c0 < dst.ne[0]) *reinterpret_cast<float4 *>(out + c0) = *reinterpret_cast<const float4 *>(row + c0);
+        return;
+    }
+    for (int e = 0; e < 4; e++) if (c0 + e < dst.ne[0]) out[c0 + e] = ok ? row[c0 + e] : __int_as_float(0x7fc00000);
 }
 
 // ------------------------------------------------------------------------------------------------ SOFT_MAX
@@ -936,7 +957,10 @@ extern "C" int b200_op_unary(int op, const b200_tensor *x, const b200_tensor *ds
     REQUIRE(op >= 0 && op <= B200_UN_RELU_SQR, B200_ERR_INVALID, "b200_op_unary: bad op %d", op);
     const int64_t n = nelements(x);
     if (n == 0) return B200_OK;
-    unary_kernel<<<grid1d(n, 256), 256, 0, (cudaStream_t)stream>>>(op, (const float *)x->data, (float *)dst->data, n, p0, p1);
+    if (n % 4 == 0 && (((uintptr_t)x->data | (uintptr_t)dst->data) & 15) == 0)
+        unary4_kernel<<<grid1d(n / 4, 256), 256, 0, (cudaStream_t)stream>>>(op, (const float4 *)x->data, (float4 *)dst->data, n / 4, p0, p1);
+    else
+        unary_kernel<<<grid1d(n, 256), 256, 0, (cudaStream_t)stream>>>(op, (const float *)x->data, (float *)dst->data, n, p0, p1);
     B200_CUDA_TRY(cudaGetLastError());
     return B200_OK;
 }
@@ -1069,6 +1093,12 @@ extern "C" int b200_op_get_rows(const b200_tensor *src, const b200_tensor *ids, 
     REQUIRE(dst->ne[0] == src->ne[0] && dst->ne[1] == ids->ne[0], B200_ERR_INVALID, "b200_op_get_rows: shape mismatch");
     if (nelements(dst) == 0) return B200_OK;
     REQUIRE(ids->ne[1] <= 65535 && ids->ne[2] <= 65535, B200_ERR_UNSUPPORTED, "b200_op_get_rows: too many index rows");
+    if (t == B200_TYPE_F32 && ids->ne[1] == 1 && ids->ne[2] == 1 && ids->ne[0] <= 65535) {
+        const bool vec4 = dst->ne[0] % 4 == 0 && (((uintptr_t)src->data | src->nb[1] | (uintptr_t)dst->data | dst->nb[1]) & 15) == 0;
+        get_rows_f32_kernel<<<dim3((unsigned)((dst->ne[0] + 1023) / 1024), (unsigned)ids->ne[0]), 256, 0, (cudaStream_t)stream>>>(td(src), td(ids), td(dst), vec4);
+        B200_CUDA_TRY(cudaGetLastError());
+        return B200_OK;
+    }
     dim3 grid((unsigned)ids->ne[0], (unsigned)ids->ne[1], (unsigned)ids->ne[2]);
     get_rows_kernel<<<grid, 256, 0, (cudaStream_t)stream>>>(td(src), t, td(ids), td(dst));
     B200_CUDA_TRY(cudaGetLastError());

@@ -124,6 +124,50 @@ __global__ void __launch_bounds__(1024) norm_reg_kernel(TD x, const float *__res
     }
 }
 
+// Short rows (the heads of a mixer's read-out): a warp per row, NW_WARPS rows per CTA, no barrier.  Row numbers fit 32 bits.
+constexpr int NW_WARPS = 8;
+__device__ __forceinline__ char *row_ptr32(const TD &t, unsigned r) {
+    const unsigned n1 = (unsigned)t.ne[1], n2 = (unsigned)t.ne[2], q = r / n1, i3 = q / n2;
+    return t.data + (int64_t)(r - q * n1) * t.nb[1] + (int64_t)(q - i3 * n2) * t.nb[2] + (int64_t)i3 * t.nb[3];
+}
+template <int KIND, bool GATE, int VPT>
+__global__ void __launch_bounds__(NW_WARPS * 32) norm_warp_kernel(TD x, const float *__restrict__ w, unsigned w_period, const float *__restrict__ bias, TD gate,
+                                                                  const float *__restrict__ gate_bias, int gate_out, TD res, bool has_res, TD dst, float eps, unsigned rows) {
+    const unsigned r = blockIdx.x * NW_WARPS + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31, n = (int)x.ne[0];
+    if (r >= rows) return;
+    const float *xr = (const float *)row_ptr32(x, r), *gr = GATE ? (const float *)row_ptr32(gate, r) : nullptr, *rr = has_res ? (const float *)row_ptr32(res, r) : nullptr;
+    const float *wr = w ? w + (int64_t)(r % w_period) * n : nullptr;
+    float *yr = (float *)row_ptr32(dst, r);
+    float v[VPT], g[VPT], s = 0.f, mean = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; k++) {
+        const int i = lane + 32 * k;
+        v[k] = i < n ? xr[i] : 0.f;
+        if (GATE) g[k] = i < n ? gr[i] + (gate_bias ? gate_bias[i] : 0.f) : 0.f;
+        if (GATE && !gate_out) v[k] *= sigmoidf_(g[k]);
+        s += KIND == B200_NORM_RMS ? v[k] * v[k] : v[k];
+    }
+    s = warp_sum(s);
+    if (KIND == B200_NORM_LAYER) {
+        mean = s / (float)n;
+        s = 0.f;
+#pragma unroll
+        for (int k = 0; k < VPT; k++) { const float d = lane + 32 * k < n ? v[k] - mean : 0.f; s += d * d; }
+        s = warp_sum(s);
+    }
+    const float scale = 1.0f / sqrtf(s / (float)n + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; k++) {
+        const int i = lane + 32 * k;
+        if (i >= n) continue;
+        float y = (v[k] - mean) * scale * (wr ? wr[i] : 1.0f);
+        if (bias) y += bias[i];
+        if (GATE && gate_out) y *= gate_out == 2 ? g[k] * sigmoidf_(g[k]) : sigmoidf_(g[k]);
+        yr[i] = y + (rr ? rr[i] : 0.f);
+    }
+}
+
 template <int VPT>
 __global__ void __launch_bounds__(1024) polynorm_reg_kernel(TD x, const float *__restrict__ coef, TD dst, float eps) {
     __shared__ float sh[32];
@@ -225,73 +269,104 @@ __global__ void __launch_bounds__(1024) norm_pair_kernel(TD x1, const float *__r
     }
 }
 
-// A sublayer's result (or the weighted sum over a token's experts and a shared one) behind its norm, the residual stream, and the
-// input norm of the next sublayer: one CTA per token, the row in registers throughout.  Everything a thread reads -- result rows,
-// residual, both norms' vectors -- is requested before the first block-wide sum (rows longer than 8 values per thread fetch the
-// second norm's vectors where they are used: registers).
+// Mean (layer norm) and 1 / sqrt(variance + eps) of the row whose values the block keeps in registers.  A warp takes its own mean and
+// the squared deviations from it, the warps' (count, mean, deviations) meet in shared memory behind ONE barrier, and every warp joins
+// them:  sum of squared deviations = sum_w (M2_w + count_w (mean_w - mean)^2).  cnt: how many of the row's values this warp holds.
 template <int VPT>
+__device__ __forceinline__ void row_statistics(const float (&v)[VPT], const bool (&ok)[VPT], bool layer, int cnt, int n, float eps, float (*sh)[32], float &mean, float &scale) {
+    const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
+    float m = 0.f, q = 0.f;
+    if (layer) {
+#pragma unroll
+        for (int k = 0; k < VPT; k++) m += v[k];  // values beyond the row are zero
+        m = warp_sum(m) / (float)(cnt > 0 ? cnt : 1);
+    }
+#pragma unroll
+    for (int k = 0; k < VPT; k++) { const float d = ok[k] ? v[k] - m : 0.f; q += d * d; }
+    q = warp_sum(q);
+    if (nw > 1) {
+        if (l == 0) { sh[0][w] = m; sh[1][w] = q; sh[2][w] = (float)cnt; }
+        __syncthreads();
+        const float mw = l < nw ? sh[0][l] : 0.f, qw = l < nw ? sh[1][l] : 0.f, cw = l < nw ? sh[2][l] : 0.f;
+        m = layer ? warp_sum(mw * cw) / (float)n : 0.f;
+        q = warp_sum(qw + (layer ? cw * (mw - m) * (mw - m) : 0.f));
+    }
+    mean = m;
+    scale = 1.0f / sqrtf(q / (float)n + eps);
+}
+
+// A sublayer's result (or the weighted sum over a token's experts and a shared one) behind its norm, the residual stream, and the
+// input norm of the next sublayer: one CTA per token, the row in registers throughout, one barrier per norm.  Everything a thread
+// reads of the row -- results, residual, the first norm's vectors -- is requested before the first barrier.  VEC: a thread owns groups
+// of 4 neighbours (16-byte accesses), else single values blockDim apart.
+template <int VPT, bool VEC>
 __global__ void __launch_bounds__(1024) norm_chain_kernel(const b200_norm_chain_args a) {
-    constexpr bool EARLY = VPT <= 4;
-    __shared__ float sh[32];
+    __shared__ float sh[2][3][32];
     const int64_t t = blockIdx.x;
-    const int n = (int)a.n;
-    float v[VPT], w1[VPT], b1[VPT], w2[VPT], b2[VPT], rv[VPT];
+    const int n = (int)a.n, bd = blockDim.x, tid = threadIdx.x;
+    auto at = [&](int k) { return VEC ? 4 * (tid + (k >> 2) * bd) + (k & 3) : tid + k * bd; };
+    float v[VPT], w1[VPT], b1[VPT], rv[VPT];
+    bool ok[VPT];
+    int cnt = 0;  // the row's values in this warp
 #pragma unroll
     for (int k = 0; k < VPT; k++) {
-        const int i = threadIdx.x + k * blockDim.x;
-        const bool ok = i < n;
-        v[k] = 0.f;
-        w1[k] = (a.w1 && ok) ? a.w1[i] : 1.f;
-        b1[k] = (a.b1 && ok) ? a.b1[i] : 0.f;
-        rv[k] = (a.res && ok) ? a.res[t * a.res_stride + i] : 0.f;
-        if (EARLY && a.h) { w2[k] = (a.w2 && ok) ? a.w2[i] : 1.f; b2[k] = (a.b2 && ok) ? a.b2[i] : 0.f; }
+        ok[k] = at(k) < n;
+        if (!VEC || (k & 3) == 0) { const int start = VEC ? 128 * (tid >> 5) + (k >> 2) * 4 * bd : 32 * (tid >> 5) + k * bd; cnt += max(0, min(VEC ? 128 : 32, n - start)); }
     }
-    for (int kk = 0; kk < a.n_y; kk++) {
-        const float wk = a.yw ? a.yw[t * a.yw_s_tok + kk] : 1.0f;
-        const float *yk = a.y + t * a.y_s_tok + kk * a.y_s_slot;
+    auto load = [&](const float *p, float none, float (&o)[VPT]) {
 #pragma unroll
-        for (int k = 0; k < VPT; k++) {
-            const int i = threadIdx.x + k * blockDim.x;
-            if (i < n) v[k] += wk * yk[i];
-        }
-    }
-#pragma unroll
-    for (int k = 0; k < VPT; k++) {
-        const int i = threadIdx.x + k * blockDim.x;
-        v[k] *= a.y_scale;
-        if (a.shared && i < n) v[k] += a.shared[t * a.shared_stride + i];
-    }
-#pragma unroll
-    for (int pass = 0; pass < 2; pass++) {
-        if (pass == 1 && !a.h) break;
-        const int kind = pass ? a.kind2 : a.kind1;
-        float mean = 0.f, ss = 0.f;
-        if (kind == B200_NORM_LAYER) {
-            float s = 0.f;
-#pragma unroll
-            for (int k = 0; k < VPT; k++) s += v[k];  // values beyond the row are zero
-            mean = block_sum(s, sh) / (float)n;
-        }
-#pragma unroll
-        for (int k = 0; k < VPT; k++) { const float d = threadIdx.x + k * blockDim.x < n ? v[k] - mean : 0.f; ss += d * d; }
-        const float scale = 1.0f / sqrtf(block_sum(ss, sh) / (float)n + a.eps);
-        if (pass == 0) {
-#pragma unroll
-            for (int k = 0; k < VPT; k++) {
-                const int i = threadIdx.x + k * blockDim.x;
-                v[k] = i < n ? rv[k] + ((v[k] - mean) * scale * w1[k] + b1[k]) : 0.f;
-                if (i < n) a.x[t * a.x_stride + i] = v[k];
-            }
-        } else {
-#pragma unroll
-            for (int k = 0; k < VPT; k++) {
-                const int i = threadIdx.x + k * blockDim.x;
-                if (i >= n) continue;
-                const float w = EARLY ? w2[k] : (a.w2 ? a.w2[i] : 1.f), b = EARLY ? b2[k] : (a.b2 ? a.b2[i] : 0.f);
-                a.h[t * a.h_stride + i] = (v[k] - mean) * scale * w + b;
+        for (int k = 0; k < VPT; k += VEC ? 4 : 1) {
+            if constexpr (VEC) {
+                float4 q = make_float4(none, none, none, none);
+                if (p && ok[k]) q = *reinterpret_cast<const float4 *>(p + at(k));
+                o[k] = q.x; o[k + 1] = q.y; o[k + 2] = q.z; o[k + 3] = q.w;
+            } else {
+                o[k] = p && ok[k] ? p[at(k)] : none;
             }
         }
+    };
+    auto store = [&](float *p, const float (&o)[VPT]) {
+#pragma unroll
+        for (int k = 0; k < VPT; k += VEC ? 4 : 1) {
+            if (!ok[k]) continue;
+            if constexpr (VEC) *reinterpret_cast<float4 *>(p + at(k)) = make_float4(o[k], o[k + 1], o[k + 2], o[k + 3]);
+            else p[at(k)] = o[k];
+        }
+    };
+    load(a.y + t * a.y_s_tok, 0.f, v);
+    load(a.w1, 1.f, w1);
+    load(a.b1, 0.f, b1);
+    load(a.res ? a.res + t * a.res_stride : nullptr, 0.f, rv);
+    if (a.yw || a.n_y > 1 || a.shared || a.y_scale != 1.0f) {
+        const float f0 = a.y_scale * (a.yw ? a.yw[t * a.yw_s_tok] : 1.0f);
+#pragma unroll
+        for (int k = 0; k < VPT; k++) v[k] *= f0;
+        for (int kk = 1; kk < a.n_y; kk++) {
+            const float fk = a.y_scale * (a.yw ? a.yw[t * a.yw_s_tok + kk] : 1.0f);
+            float u[VPT];
+            load(a.y + t * a.y_s_tok + kk * a.y_s_slot, 0.f, u);
+#pragma unroll
+            for (int k = 0; k < VPT; k++) v[k] += fk * u[k];
+        }
+        if (a.shared) {
+            float u[VPT];
+            load(a.shared + t * a.shared_stride, 0.f, u);
+#pragma unroll
+            for (int k = 0; k < VPT; k++) v[k] += u[k];
+        }
     }
+    float mean, scale;
+    row_statistics(v, ok, a.kind1 == B200_NORM_LAYER, cnt, n, a.eps, sh[0], mean, scale);
+#pragma unroll
+    for (int k = 0; k < VPT; k++) v[k] = ok[k] ? rv[k] + ((v[k] - mean) * scale * w1[k] + b1[k]) : 0.f;
+    store(a.x + t * a.x_stride, v);
+    if (!a.h) return;
+    load(a.w2, 1.f, w1);
+    load(a.b2, 0.f, b1);
+    row_statistics(v, ok, a.kind2 == B200_NORM_LAYER, cnt, n, a.eps, sh[1], mean, scale);
+#pragma unroll
+    for (int k = 0; k < VPT; k++) v[k] = (v[k] - mean) * scale * w1[k] + b1[k];
+    store(a.h + t * a.h_stride, v);
 }
 
 // position vector of sines and cosines added to every row: a thread per pair (2i, 2i + 1), the angle pos * f_i in f32
@@ -338,9 +413,13 @@ extern "C" int b200_op_norm_chain(const b200_norm_chain_args *args, b200_stream_
     const int n = (int)a.n;
     const int rb = n <= 256 ? 64 : n <= 512 ? 128 : n <= 1024 ? 256 : n <= 2048 ? 512 : 1024, vpt = (n + rb - 1) / rb;
     const cudaStream_t st = (cudaStream_t)stream;
-    if (vpt <= 4) norm_chain_kernel<4><<<(unsigned)a.n_tok, rb, 0, st>>>(a);
-    else if (vpt <= 8) norm_chain_kernel<8><<<(unsigned)a.n_tok, rb, 0, st>>>(a);
-    else norm_chain_kernel<16><<<(unsigned)a.n_tok, rb, 0, st>>>(a);
+    // 16-byte accesses when every row of every operand starts on a 16-byte boundary
+    auto al = [](const float *p, int64_t s0, int64_t s1 = 0) { return !p || ((((uintptr_t)p) & 15) == 0 && s0 % 4 == 0 && s1 % 4 == 0); };
+    const bool vec = n % 4 == 0 && al(a.y, a.y_s_tok, a.y_s_slot) && al(a.shared, a.shared_stride) && al(a.res, a.res_stride) && al(a.w1, 0) && al(a.b1, 0) && al(a.w2, 0) && al(a.b2, 0) &&
+                     al(a.x, a.x_stride) && al(a.h, a.h_stride);
+#define B200_NC(V) do { if (vec) norm_chain_kernel<V, true><<<(unsigned)a.n_tok, rb, 0, st>>>(a); else norm_chain_kernel<V, false><<<(unsigned)a.n_tok, rb, 0, st>>>(a); } while (0)
+    if (vpt <= 4) B200_NC(4); else if (vpt <= 8) B200_NC(8); else B200_NC(16);
+#undef B200_NC
     B200_CUDA_TRY(cudaGetLastError());
     return B200_OK;
 }
@@ -378,6 +457,18 @@ extern "C" int b200_op_norm_affine(const b200_tensor *x, const float *w, int64_t
     const int block = x->ne[0] >= 4096 ? 512 : (x->ne[0] >= 1024 ? 256 : 128);
     const cudaStream_t st = (cudaStream_t)stream;
     TD tg = gate ? td(gate) : td(x), tr = res ? td(res) : td(x);
+    if (x->ne[0] <= 256 && rows <= 0x7fffffff && w_period <= 0x7fffffff) {  // short rows: a warp each
+        const int n = (int)x->ne[0];
+#define B200_NORM_WARP(K, G, V) norm_warp_kernel<K, G, V><<<(unsigned)((rows + NW_WARPS - 1) / NW_WARPS), NW_WARPS * 32, 0, st>>>(td(x), w, (unsigned)w_period, bias, tg, gate_bias, gate_out, tr, \
+                                                                                                                      res != nullptr, td(dst), eps, (unsigned)rows)
+#define B200_NORM_WARP_V(K, G) do { if (n <= 64) B200_NORM_WARP(K, G, 2); else if (n <= 128) B200_NORM_WARP(K, G, 4); else B200_NORM_WARP(K, G, 8); } while (0)
+        if (kind == B200_NORM_RMS) { if (gate) B200_NORM_WARP_V(B200_NORM_RMS, true); else B200_NORM_WARP_V(B200_NORM_RMS, false); }
+        else { if (gate) B200_NORM_WARP_V(B200_NORM_LAYER, true); else B200_NORM_WARP_V(B200_NORM_LAYER, false); }
+#undef B200_NORM_WARP_V
+#undef B200_NORM_WARP
+        B200_CUDA_TRY(cudaGetLastError());
+        return B200_OK;
+    }
     if (x->ne[0] <= 16384) {  // the row fits the registers of one block
         const int n = (int)x->ne[0];
         const int rb = n <= 256 ? 64 : n <= 1024 ? 128 : n <= 2048 ? 256 : n <= 4096 ? 512 : 1024;

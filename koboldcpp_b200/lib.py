@@ -157,6 +157,7 @@ class TimeMixArgs(C.Structure):
 _SIGS = {
     # name: (restype, argtypes)
     "b200_last_error": (C.c_char_p, []),
+    "b200_gemm_status": (C.c_int, []),
     "b200_version": (C.c_char_p, []),
     "b200_set_pdl": (None, [C.c_int]),
     "b200_device_count": (C.c_int, []),
