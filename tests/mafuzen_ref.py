@@ -248,3 +248,136 @@ def forward(cfg, weights, tokens, state=None, want_layers=False):
 
 def logits(cfg, weights, tokens):
     return forward(cfg, weights, tokens)[0]
+
+
+# ------------------------------------------------------------------------------------------------ small random models for the tests
+def bf16_round(x):
+    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32).astype(np.uint64)
+    u = ((u + 0x7FFF + ((u >> 16) & 1)) >> 16) << 16
+    return u.astype(np.uint32).view(np.float32)
+
+
+def dense_cfg(ff=40):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe_cfg(ff=24, experts=6, top=2, shared=16):
+    m = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    if shared:
+        m["shared"] = {"ff": shared}
+    return m
+
+
+def attention_layer(heads=4, kv_heads=2, dim=16, vdim=24, scale=None, kv_from=None, mlp="moe"):
+    mx = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale if scale is not None else 1.0 / math.sqrt(dim)}
+    if kv_from is not None:
+        mx["kv_from"] = kv_from
+    return {"type": "attention", "mixer": mx, "mlp": moe_cfg() if mlp == "moe" else mlp}
+
+
+def retention_layer(heads=3, dim=16, vdim=20, rot=8, base=1000.0, decay=None, mlp="moe"):
+    return {"type": "retention", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "rot": {"dims": rot, "base": base},
+                                           "decay": decay or [1.0 - 2.0 ** (-2 - i) for i in range(heads)]}, "mlp": moe_cfg() if mlp == "moe" else mlp}
+
+
+def parallel_layer(heads=4, kv_heads=2, dim=16, size=11, keep_first=3, scale=None, mix_heads=3, mix_dim=12, left_scale=0.7, right_scale=1.3, mlp="moe"):
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": size, "keep_first": keep_first}, "scale": scale if scale is not None else 1.0 / math.sqrt(dim)}
+    return {"type": "parallel", "mixer": {"left": left, "left_scale": left_scale, "right": {"heads": mix_heads, "dim": mix_dim}, "right_scale": right_scale},
+            "mlp": moe_cfg() if mlp == "moe" else mlp}
+
+
+def make_config(layers, width=40, vocab=61, eps=1e-5, embed_scale=3.0, side=12):
+    return {"architecture": "Mafuzen", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": embed_scale},
+            "token_side": {"dim": side} if side else None, "layers": layers}
+
+
+def random_weights(cfg, seed=0, rank=5):
+    """name -> float64 arrays whose values bfloat16 holds exactly (tables: int32), so that the served (bf16) and the exact (f32) modes
+    read the same model."""
+    rng = np.random.default_rng(seed)
+    Wd, Vc = cfg["width"], cfg["vocab"]
+    W = {}
+
+    def mat(name, rows, cols, g=1.0):
+        W[name] = bf16_round(rng.standard_normal((rows, cols)) * g / math.sqrt(cols)).astype(np.float64)
+
+    def vec(name, n, mean=0.0, spread=0.3):
+        W[name] = bf16_round(mean + spread * rng.standard_normal(n)).astype(np.float64)
+
+    def norm(name):
+        vec(name, Wd, 1.0, 0.2)
+        vec(name + ".b", Wd, 0.0, 0.2)
+
+    W["embed"] = bf16_round(rng.standard_normal((Vc, Wd)) / math.sqrt(Wd) * 3.0).astype(np.float64)
+    norm("final.norm")
+    side = (cfg.get("token_side") or {}).get("dim", 0)
+    if side:
+        W["side.embed"] = bf16_round(rng.standard_normal((Vc, side * len(cfg["layers"])))).astype(np.float64)
+    for il, L in enumerate(cfg["layers"]):
+        p, mx = f"l{il}.", L["mixer"]
+        norm(p + "norm1")
+        norm(p + "norm1b")
+        if L["type"] == "attention":
+            H, G, D, V = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
+            mat(p + "mix.q", H * D, Wd, 1.5)
+            if mx.get("kv_from") is None:
+                mat(p + "mix.k", G * D, Wd, 1.5)
+                mat(p + "mix.v", G * V, Wd, 1.5)
+            mat(p + "mix.o", Wd, H * V)
+        elif L["type"] == "retention":
+            H, D, V = mx["heads"], mx["dim"], mx["vdim"]
+            for leaf, rows in (("q", H * D), ("k", H * D), ("v", H * V), ("g", H * V)):
+                mat(p + "mix." + leaf, rows, Wd, 1.5)
+            mat(p + "mix.o", Wd, H * V)
+        else:
+            a, HR, DR = mx["left"], mx["right"]["heads"], mx["right"]["dim"]
+            H, G, D = a["heads"], a["kv_heads"], a["dim"]
+            mat(p + "mix.left.q", H * D, Wd, 1.5)
+            mat(p + "mix.left.k", G * D, Wd, 1.5)
+            mat(p + "mix.left.g", H * D, Wd, 1.5)
+            mat(p + "mix.left.o", Wd, H * D)
+            for s in "rkvgw":
+                vec(p + "mix.right.mu." + s, Wd, 0.5, 0.3)
+            for s in "rkvg":
+                mat(p + "mix.right." + s, HR * DR, Wd, 1.5)
+            mat(p + "mix.right.w1", rank, Wd, 1.0)
+            mat(p + "mix.right.w2", HR * DR, rank, 1.0)
+            vec(p + "mix.right.w0", HR * DR, -2.0, 1.5)
+            W[p + "mix.right.u"] = bf16_round(rng.standard_normal((HR, DR))).astype(np.float64)
+            vec(p + "mix.right.norm", HR * DR, 1.0, 0.3)
+            mat(p + "mix.right.o", Wd, HR * DR)
+        if side:
+            mat(p + "side.gate", side, Wd, 1.5)
+            mat(p + "side.proj", Wd, side)
+            vec(p + "side.norm", Wd, 0.7, 0.3)
+        mlp = L.get("mlp")
+        if mlp is None:
+            continue
+        norm(p + "norm2")
+        norm(p + "norm2b")
+        if mlp["kind"] == "dense":
+            mat(p + "mlp.gate", mlp["ff"], Wd, 1.5)
+            mat(p + "mlp.up", mlp["ff"], Wd, 1.5)
+            mat(p + "mlp.down", Wd, mlp["ff"])
+            continue
+        F, E, top = mlp["expert"]["ff"], mlp["router"]["experts"], mlp["router"]["top"]
+        W[p + "mlp.table"] = np.stack([rng.permutation(E)[:top] for _ in range(Vc)]).astype(np.int32)
+        for e in range(E):
+            mat(p + f"mlp.e{e}.up", F, Wd, 1.5)
+            mat(p + f"mlp.e{e}.down", Wd, F, 1.5)
+        if mlp.get("shared"):
+            mat(p + "mlp.shared.up", mlp["shared"]["ff"], Wd, 1.5)
+            mat(p + "mlp.shared.down", Wd, mlp["shared"]["ff"], 1.5)
+    return W
+
+
+def as_tensors(W):
+    """name -> (dtype, shape, raw bytes), the form the loader takes: matrices and vectors as bf16 bits, tables as int32."""
+    out = {}
+    for name, a in W.items():
+        if a.dtype == np.int32:
+            out[name] = ("I32", tuple(a.shape), np.ascontiguousarray(a).reshape(-1).view(np.uint8))
+            continue
+        bits = (np.ascontiguousarray(a, dtype=np.float32).view(np.uint32) >> 16).astype(np.uint16)
+        out[name] = ("BF16", tuple(a.shape), bits.view(np.uint8).reshape(-1))
+    return out
