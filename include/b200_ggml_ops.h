@@ -117,18 +117,21 @@ enum b200_ext_op {
     B200_EXT_ROPE_TABLE = 3,   /* src: x, pos, freqs; in place; op_params: [2] n_dims, [3] mscale, [4] neox */
     B200_EXT_WEIGHTED_SUM = 4, /* src: xs [n, J], w [J] */
     B200_EXT_SIGMOID_MUL = 5,  /* src: a, b: dst = a * sigmoid(b), any strides */
-    B200_EXT_LATENT_KV_STORE = 6, /* src: dkv, norm w, pos, freqs, cells, cache; op_params: [2] kv_rank, [3] eps, [4] mscale, [5] n_dims */
-    B200_EXT_LATENT_ATTN = 7,  /* src: q_lat, q_rot, cache, sink, tok_seq, tok_pos, cell_seq, cell_pos; op_params: [2] kv_rank, [3] scale, [4] window */
+    B200_EXT_LATENT_KV_STORE = 6, /* src: dkv, norm w, pos, freqs, cells, cache, [query latent [q_rank, T], its norm w: RMS-normed in place]; op_params: [2] kv_rank, [3] eps,
+                                  [4] mscale, [5] n_dims; freqs may be NULL without rotation */
+    B200_EXT_LATENT_ATTN = 7,  /* src: q_lat, q_rot, cache, sink, tok_seq, tok_pos, cell_seq, cell_pos, [head gate [heads, T]]; op_params: [2] kv_rank, [3] scale, [4] window,
+                                  [5] bf16 products */
     B200_EXT_MLSTM_SCAN = 8,   /* src: q, k, v, ig, fg, i_bias, f_bias, seq_info, state; op_params: [2] heads, [3] dim, [4] vdim, [5] gate_cap */
     B200_EXT_QKV_STORE = 9,    /* src: q, k, v, vecs (the present ones of q.b, k.b, v.b, q.norm, k.norm packed in one tensor, or NULL), pos, freqs,
                                   cells, k cache, v cache; q in place; op_params: [2] dim, [3] vdim, [4] n_dims, [5] eps, [6] biases present, [7] norms present
                                   (1: over the whole row, 2: per head with one weight vector of dim values, 3: per head without a weight), [8] pairs are (i, i + n_dims / 2), [9] every head of v is divided
-                                  by its root mean square, [10] q temperature coefficient, [11] its period in positions; freqs may be NULL without rotation */
+                                  by its root mean square, [10] q temperature coefficient, [11] its period in positions, [12] factor on sine and cosine (0 reads as 1);
+                                  freqs may be NULL without rotation */
     B200_EXT_SINK_ATTN = 10,   /* src: q, k cache, v cache, sink, tok_seq, tok_pos, cell_seq, cell_pos, [head gate [heads, T]]; op_params: [2] dim, [3] scale,
                                   [4] window, [5] keep_first, [6] bf16 products, [7] vdim, [8] chunk, [9] enum b200_attn_weights, [10] linear distance bias, [11] factor on
-                                  the result (0 reads as 1); src[8] of [heads * vdim, T]: a gate per value; src[9]: score bias by distance [n_dist, heads] (optional) */
-    B200_EXT_LINEAR_ATTN_SCAN = 11, /* src: q, k, v, decay, seq_info, state, [pos, freqs]; op_params: [2] heads, [3] dim, [4] vdim, [5] silu on q / k / v, [6] factor on k
-                                  (0 reads as 1), [7] n_dims of the rotation (0: none) */
+                                  the result (0 reads as 1), [12] soft cap of the scores (0: none); src[8] of [heads * vdim, T]: a gate per value; src[9]: score bias by distance [n_dist, heads] (optional) */
+    B200_EXT_LINEAR_ATTN_SCAN = 11, /* src: q, k, v, decay [heads] (or NULL), seq_info, state, [pos, freqs], [z [heads * dim, T], its bias]: a decay per token and key channel; op_params: [2] heads, [3] dim, [4] vdim, [5] silu on q / k / v, [6] factor on k
+                                  (0 reads as 1), [7] n_dims of the rotation (0: none), [8] tau of the decay per channel */
     B200_EXT_MOE_ROUTE = 12,   /* src: logits, correction; dst [2 n_used, T]: per token n_used weights (f32), then n_used expert ids (i32);
                                   op_params: [2] n_group, [3] n_group_used, [4] scale, [5] n_used, [6] enum b200_router_score, [7] weights are the
                                   scores as they are (no division by their sum) */
@@ -143,7 +146,7 @@ enum b200_ext_op {
     B200_EXT_SHORT_CONV = 18,  /* src: x [channels, T], w [taps, channels], bias (optional), seq_info, tail [(taps - 1) * channels, slots]; op_params: [2] activation
                                   (0 none, 1 silu) */
     B200_EXT_DELTA_RULE_SCAN = 19, /* src: q, k, v, a, b, a_log, dt_bias, seq_info, state; op_params: [2] heads, [3] kv_heads, [4] dim, [5] vdim, [6] q and k become
-                                  unit vectors, [7] the eps of that, [8] q scale */
+                                  unit vectors, [7] the eps of that, [8] q scale; a and dt_bias of heads * dim values: a decay per key channel */
     B200_EXT_MINGRU_SCAN = 20, /* src: z, x, g (optional), z bias, x bias (optional), seq_info, state [width, slots] */
     B200_EXT_NORM_PAIR = 21,   /* src: x1, w1, b1 (optional), x2, w2: dst = N(x1 + b1) * w1 + N(x2) * w2, N the RMS norm; op_params: [3] eps */
     B200_EXT_NORM_CHAIN = 22,  /* src: y [n, n_y, T], y weights [n_y, T] (optional), shared [n, T] (optional), res [n, T] (optional), w1, b1, w2, b2 (optional each);
@@ -159,7 +162,11 @@ enum b200_router_score { B200_ROUTER_SIGMOID = 0, B200_ROUTER_SOFTMAX = 1 /* ove
 /* gated activations dst = f(a, b): SILU a sigmoid(a) b; GELU_TANH gelu(a) b with the tanh form of gelu; SWISH_CLAMPED with g = min(a, limit),
  * u = clamp(b, -limit, limit): g sigmoid(alpha g) (u + 1) */
 enum b200_glu_kind { B200_GLU_SILU = 0, B200_GLU_GELU_TANH = 1, B200_GLU_SWISH_CLAMPED = 2 };
-enum b200_norm_kind { B200_NORM_LAYER = 0 /* (x - mean) / sqrt(var + eps) */, B200_NORM_RMS = 1 /* x / sqrt(mean(x^2) + eps) */ };
+enum b200_norm_kind {
+    B200_NORM_LAYER = 0, /* (x - mean) / sqrt(var + eps) */
+    B200_NORM_RMS = 1,   /* x / sqrt(mean(x^2) + eps) */
+    B200_NORM_NONE = 2,  /* x (the first step of b200_op_norm_chain only): a residual connection without a norm behind the sublayer */
+};
 
 /* dst[row] = (res ? res[row] : 0) + N(x[row] * (gate ? sigmoid(gate[row] + gate_bias) : 1)) * w[(row % w_period)], N the layer
  * norm or the RMS norm over ne0.  x, gate, res, dst: f32 rows (nb[0] == 4), any row strides; w: [w_period][ne0] f32 or NULL;
@@ -181,7 +188,7 @@ B200_API int b200_op_norm_pair(const b200_tensor *x1, const float *w1, const flo
 /* A sublayer's result behind its norm, the residual stream, and the next sublayer's input norm in one launch, a token per CTA:
  *   s = y_scale * sum_k yw[t][k] * y[t][k] + shared[t]      (yw NULL: weights of one; shared optional; n_y = 1 for a plain result)
  *   x[t] = res[t] + N1(s) * w1 + b1,   h[t] = N2(x[t]) * w2 + b2   (h NULL: not wanted)
- * N1, N2: enum b200_norm_kind with the same eps; w1, b1, w2, b2, res optional.  Strides in floats; n <= 16384. */
+ * N1, N2: enum b200_norm_kind with the same eps (N1 may be B200_NORM_NONE); w1, b1, w2, b2, res optional.  Strides in floats; n <= 16384. */
 typedef struct {
     const float *y; int64_t y_s_slot, y_s_tok;
     const float *yw; int64_t yw_s_tok;
@@ -219,12 +226,19 @@ B200_API int b200_op_latent_kv_store(const float *dkv, int64_t dkv_stride, const
                                      float *cache, int64_t cache_stride, int32_t kv_rank, int32_t rot_dim, int32_t n_dims, float mscale, float eps,
                                      int32_t n_tokens, b200_stream_t stream);
 
+/* The same, and in the same launch the query latents q [n_tokens][q_rank] are RMS-normed with q_w in place (q NULL: none).  pos and freqs may
+ * be NULL when n_dims is 0. */
+B200_API int b200_op_latent_store(const float *dkv, int64_t dkv_stride, const float *w, const int32_t *pos, const float *freqs, const int32_t *cells,
+                                  float *cache, int64_t cache_stride, int32_t kv_rank, int32_t rot_dim, int32_t n_dims, float mscale, float eps,
+                                  float *q, int64_t q_stride, const float *q_w, int32_t q_rank, int32_t n_tokens, b200_stream_t stream);
+
 /* Attention of H query heads over the latent cache (every head reads the same rows: the key is the whole row, the value its
  * first kv_rank entries).  score = scale * (q_lat . row[:kv_rank] + q_rot . row[kv_rank:]); a token sees the cells of its own
  * sequence with cell_pos <= tok_pos (and cell_pos > tok_pos - window when window > 0); softmax in f32 whose denominator also
  * holds exp(sink[h]) when sink != NULL.  Strides are in floats.  dst[h][t][:kv_rank] = sum_c p_c row_c[:kv_rank].
  * bf16_products != 0 allows the two contractions of a prompt batch (16 tokens or more) to take queries, rows and weights rounded
- * to bf16 with f32 accumulation (scores, maxima, exponentials and sums stay f32); 0 keeps every product in f32. */
+ * to bf16 with f32 accumulation (scores, maxima, exponentials and sums stay f32); 0 keeps every product in f32.  gate != NULL: the
+ * result of head h of token t is multiplied by sigmoid(gate[t * gate_stride + h]). */
 typedef struct {
     const float *q_lat; int64_t q_lat_s_head, q_lat_s_tok;
     const float *q_rot; int64_t q_rot_s_head, q_rot_s_tok;
@@ -235,6 +249,7 @@ typedef struct {
     int32_t kv_rank, rot_dim, n_head, n_tokens, n_kv, window;
     float scale;
     int32_t bf16_products;
+    const float *gate; int64_t gate_stride;
 } b200_latent_attn_args;
 B200_API int b200_op_latent_attn(const b200_latent_attn_args *a, b200_stream_t stream);
 
@@ -291,10 +306,11 @@ typedef struct {
     float   q_temp_coef;                   /* != 0: q is multiplied by 1 + coef * ln(floor((pos + 1) / q_temp_every) + 1) */
     int32_t q_temp_every;
     int32_t qk_unit_rms;                   /* 1: every head of q and k is divided by sqrt(mean(x^2) + eps), no weight */
+    float   rope_mscale;                   /* sine and cosine are multiplied by this (0 reads as 1) */
 } b200_qkv_store_args;
 B200_API int b200_op_qkv_store(const b200_qkv_store_args *a, b200_stream_t stream);
 
-/* score = scale * q . k (+ dist_bias, see below); a token sees the cells of its own sequence with cell_pos <= tok_pos and (window == 0 or
+/* score = scale * q . k, soft-capped when softcap > 0 (softcap * tanh(score / softcap)) (+ dist_bias, see below); a token sees the cells of its own sequence with cell_pos <= tok_pos and (window == 0 or
  * tok_pos - cell_pos < window or cell_pos < keep_first) and (chunk == 0 or tok_pos / chunk == cell_pos / chunk: positions are cut
  * into chunks counted from 0 and nothing is seen across a cut); softmax in f32 whose denominator also holds exp(sink[h]) when
  * sink != NULL (the sink has no key and no value).  gate != NULL: head h of token t is multiplied by sigmoid(gate[t * gate_stride
@@ -316,6 +332,7 @@ typedef struct {
     int32_t dist_linear;                   /* 1: dist_bias[h][0] is a bias per position instead: dist_bias[h][0] * (tok_pos - cell_pos) joins the score */
     int32_t gate_per_value;                /* 1: gate has n_head * vdim values per token, one for every value of the result */
     float   out_scale;                     /* the result is multiplied by this (0 reads as 1) */
+    float   softcap;                       /* > 0: the scaled score s becomes softcap * tanh(s / softcap) */
 } b200_sink_attn_args;
 B200_API int b200_op_sink_attn(const b200_sink_attn_args *a, b200_stream_t stream);
 /* The same with a workspace of b200_sink_attn_workspace_bytes(a) bytes (16-byte aligned; 0: none needed): with few tokens and
@@ -336,6 +353,8 @@ typedef struct {
     float   k_scale;                       /* k is multiplied by this (0 reads as 1) */
     const int32_t *pos; const float *freqs; /* n_dims > 0: entry i of every head of q and k turns with entry i + n_dims / 2 by pos[t] * freqs[i], */
     int32_t n_dims;                        /* i < n_dims / 2, behind the activation; entries from n_dims on stay (every CTA of a head turns its own copy: for few tokens) */
+    const float *z; int64_t z_stride;      /* [n_tokens][heads * dim], instead of decay[h]: key channel d of head h forgets by sigmoid(z + z_bias)^(1 / tau) per token */
+    const float *z_bias; float tau;        /* [heads * dim] or NULL; tau > 0 */
 } b200_linear_attn_args;
 B200_API int b200_op_linear_attn_scan(const b200_linear_attn_args *a, b200_stream_t stream);
 
@@ -402,12 +421,13 @@ B200_API int b200_op_short_conv(const b200_short_conv_args *a, b200_stream_t str
 typedef struct {
     const float *q, *k, *v; int64_t q_stride, k_stride, v_stride;  /* q, k [n_tokens][kv_heads * dim], v [n_tokens][heads * vdim] */
     const float *a, *b; int64_t a_stride, b_stride;                /* [n_tokens][heads] */
-    const float *a_log, *dt_bias;                                  /* [heads] */
+    const float *a_log, *dt_bias;                                  /* [heads]; dt_bias may be NULL */
     const int32_t *seq_info; int32_t n_seq;
     float *state; int64_t slot_stride;
     float *dst; int64_t dst_stride;                                /* [n_tokens][heads * vdim] */
     int32_t heads, kv_heads, dim, vdim, unit_qk;
     float unit_eps, q_scale;
+    int32_t channel_decay;                                         /* 1: a is [n_tokens][heads * dim] and dt_bias [heads * dim]: g per key channel (row of S) */
 } b200_delta_rule_args;
 B200_API int b200_op_delta_rule_scan(const b200_delta_rule_args *a, b200_stream_t stream);
 

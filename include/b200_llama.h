@@ -45,9 +45,10 @@ typedef struct {
     float   logit_softcap;           /* > 0: logits = cap * tanh(logits / cap) (architectures with their own graph) */
     float   embed_scale;             /* the embedding row is multiplied by this (0 reads as 1) */
     float   residual_mult;           /* architectures that scale a sublayer's result before it joins the residual stream (0 reads as 1) */
+    float   logit_scale;             /* the logits are multiplied by this (0 reads as 1) */
 } b200_llama_params;
 
-enum b200_arch { B200_ARCH_LLAMA = 0, B200_ARCH_GENESUN = 1, B200_ARCH_GALIRAX = 2, B200_ARCH_ZEVOPEL = 3, B200_ARCH_MEDODRA = 4, B200_ARCH_MAFUZEN = 5 };
+enum b200_arch { B200_ARCH_LLAMA = 0, B200_ARCH_GENESUN = 1, B200_ARCH_GALIRAX = 2, B200_ARCH_ZEVOPEL = 3, B200_ARCH_MEDODRA = 4, B200_ARCH_MAFUZEN = 5, B200_ARCH_TUGEZEN = 6 };
 enum b200_mixer {
     B200_MIXER_LATENT_ATTENTION = 1, B200_MIXER_MLSTM = 2,
     B200_MIXER_ATTENTION = 3, /* softmax attention of heads over kv_heads cached keys / values, per-head sink, optional window */
@@ -56,6 +57,8 @@ enum b200_mixer {
     B200_MIXER_SIGMOID_ATTENTION_GRU = 6, /* two mixers side by side: attention with sigmoid weights and a distance bias, and a minGRU */
     B200_MIXER_RETENTION = 7, /* linear attention with a fixed decay per head, rotated queries and keys, a norm per head and a gate behind it */
     B200_MIXER_WINDOW_ATTENTION_TIME_MIX = 8, /* two mixers side by side: windowed attention whose values are its keys, and time mixing */
+    B200_MIXER_GATED_LINEAR_ATTENTION = 9, /* linear attention whose state forgets by a learned decay per token and key channel */
+    B200_MIXER_ATTENTION_DELTA = 10, /* two mixers side by side: soft-capped attention, and the gated delta rule with a decay per key channel */
 };
 enum b200_mlp {
     B200_MLP_NONE = 0, B200_MLP_DENSE_POLYNORM = 1, B200_MLP_MOE_GATED = 2 /* routed gated experts */,
@@ -120,10 +123,15 @@ typedef struct {
                                         x0 being the stream as the embedding left it: the first layer of a looped stretch */
     /* attention, further switches (kv_from serves B200_MIXER_ATTENTION too: the layer has queries only and reads that layer's cache) */
     float   dist_slope_exp;          /* > 0: slope_h * distance is taken off the score, slope_h = 2^(-dist_slope_exp (h + 1) / heads) */
-    /* B200_MIXER_WINDOW_ATTENTION_TIME_MIX: heads .. keep_first describe the attention; time mixing has heads of its own */
+    /* B200_MIXER_WINDOW_ATTENTION_TIME_MIX, B200_MIXER_ATTENTION_DELTA: heads .. keep_first describe the attention; the other side has heads of its own */
     int32_t mix_heads, mix_dim;
     float   left_scale, right_scale; /* factors on the two results before they are added */
     int32_t token_side;              /* > 0: a second embedding of this size per layer joins behind the feed-forward ("side.*") */
+    float   attn_softcap;            /* > 0: an attention score s becomes softcap * tanh(s / softcap) */
+    int32_t mix_kv_heads, mix_vdim;  /* B200_MIXER_ATTENTION_DELTA: query / key heads (value head h reads h / (mix_heads / mix_kv_heads)) and value size */
+    /* low-rank projections W2 (W1 x): rows of W1 ("a1" feeds the decay per key channel, "g1" the gate per value) */
+    int32_t decay_rank, gate_rank;
+    float   decay_tau;               /* B200_MIXER_GATED_LINEAR_ATTENTION: the decay is sigmoid(z)^(1 / tau) */
 } b200_layer_params;
 
 

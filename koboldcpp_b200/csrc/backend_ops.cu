@@ -61,11 +61,12 @@ static bool ext_op_supported(const ggml_tensor *op) {
         case B200_EXT_SIGMOID_MUL:
             return s[0] && s[1] && s[0]->type == GGML_TYPE_F32 && s[1]->type == GGML_TYPE_F32 && op->type == GGML_TYPE_F32 && same_shape(s[0], op) && same_shape(s[1], op);
         case B200_EXT_LATENT_KV_STORE:
-            return f32_rows(s[0]) && f32_vec(s[1]) && i32_vec(s[2]) && f32_vec(s[3]) && i32_vec(s[4]) && f32_rows(s[5]) && op->op_params[2] > 0 &&
-                   s[0]->ne[0] == s[5]->ne[0] && op->op_params[2] <= s[0]->ne[0];
+            return f32_rows(s[0]) && f32_vec(s[1]) && i32_vec(s[2]) && (s[3] ? f32_vec(s[3]) : op->op_params[5] == 0) && i32_vec(s[4]) && f32_rows(s[5]) && op->op_params[2] > 0 &&
+                   s[0]->ne[0] == s[5]->ne[0] && op->op_params[2] <= s[0]->ne[0] && (!s[6] || (f32_rows(s[6]) && s[6]->ne[1] == s[0]->ne[1] && f32_vec(s[7]) && s[7]->ne[0] == s[6]->ne[0]));
         case B200_EXT_LATENT_ATTN:
             return f32_rows(s[0]) && (!s[1] || f32_rows(s[1])) && f32_rows(s[2]) && (!s[3] || f32_vec(s[3])) && i32_vec(s[4]) && i32_vec(s[5]) && i32_vec(s[6]) && i32_vec(s[7]) &&
-                   f32_rows(op) && op->op_params[2] == s[0]->ne[0] && op->ne[0] == s[0]->ne[0] && s[0]->ne[0] <= 1024 && s[2]->ne[0] - s[0]->ne[0] <= 128;
+                   f32_rows(op) && op->op_params[2] == s[0]->ne[0] && op->ne[0] == s[0]->ne[0] && s[0]->ne[0] <= 1024 && s[2]->ne[0] - s[0]->ne[0] <= 128 &&
+                   (!s[8] || (f32_rows(s[8]) && s[8]->ne[0] == s[0]->ne[1] && s[8]->ne[1] == s[0]->ne[2]));
         case B200_EXT_MLSTM_SCAN:
             for (int i = 0; i < 5; i++) if (!f32_rows(s[i])) return false;
             return (!s[5] || f32_vec(s[5])) && (!s[6] || f32_vec(s[6])) && i32_vec(s[7]) && f32_rows(s[8]) && f32_rows(op) && op->op_params[3] <= 512;
@@ -79,8 +80,8 @@ static bool ext_op_supported(const ggml_tensor *op) {
                    (!s[8] || (f32_rows(s[8]) && (s[8]->ne[0] == s[0]->ne[0] / op->op_params[2] || s[8]->ne[0] == s[0]->ne[0] / op->op_params[2] * op->op_params[7]) && s[8]->ne[1] == s[0]->ne[1])) &&
                    (!s[9] || (f32_vec(s[9]) && s[9]->ne[1] == s[0]->ne[0] / op->op_params[2] && s[9]->ne[0] > 0));
         case B200_EXT_LINEAR_ATTN_SCAN:
-            return f32_rows(s[0]) && f32_rows(s[1]) && f32_rows(s[2]) && f32_vec(s[3]) && i32_vec(s[4]) && f32_rows(s[5]) && f32_rows(op) && op->op_params[3] <= 256 &&
-                   (op->op_params[7] == 0 || (i32_vec(s[6]) && f32_vec(s[7])));
+            return f32_rows(s[0]) && f32_rows(s[1]) && f32_rows(s[2]) && (s[8] ? f32_rows(s[8]) && s[8]->ne[0] == s[0]->ne[0] && (!s[9] || f32_vec(s[9])) : f32_vec(s[3])) &&
+                   i32_vec(s[4]) && f32_rows(s[5]) && f32_rows(op) && op->op_params[3] <= 256 && (op->op_params[7] == 0 || (i32_vec(s[6]) && f32_vec(s[7])));
         case B200_EXT_MOE_ROUTE:
             return f32_rows(s[0]) && (!s[1] || f32_vec(s[1])) && f32_rows(op) && s[0]->ne[0] <= 256 && op->op_params[5] > 0 && op->op_params[5] <= 32 && op->ne[0] == 2 * op->op_params[5] &&
                    op->ne[1] == s[0]->ne[1];
@@ -109,7 +110,8 @@ static bool ext_op_supported(const ggml_tensor *op) {
         case B200_EXT_DELTA_RULE_SCAN:
             for (int i = 0; i < 5; i++) if (!f32_rows(s[i])) return false;
             return f32_vec(s[5]) && (!s[6] || f32_vec(s[6])) && i32_vec(s[7]) && f32_rows(s[8]) && f32_rows(op) && op->op_params[4] > 0 && op->op_params[4] <= 256 &&
-                   op->op_params[3] > 0 && op->op_params[2] % op->op_params[3] == 0;
+                   op->op_params[3] > 0 && op->op_params[2] % op->op_params[3] == 0 && (s[3]->ne[0] == op->op_params[2] || s[3]->ne[0] == (int64_t)op->op_params[2] * op->op_params[4]) &&
+                   (!s[6] || nelements(s[6]) == s[3]->ne[0]);
         case B200_EXT_MINGRU_SCAN:
             return f32_rows(s[0]) && f32_rows(s[1]) && (!s[2] || f32_rows(s[2])) && (!s[3] || f32_vec(s[3])) && (!s[4] || f32_vec(s[4])) && i32_vec(s[5]) && f32_rows(s[6]) &&
                    f32_rows(op) && s[6]->ne[0] >= op->ne[0];
@@ -145,7 +147,7 @@ static void fill_sink_attn_args(const ggml_tensor *n, b200_sink_attn_args &a) {
     if (s[8]) { a.gate = (const float *)s[8]->data; a.gate_stride = (int64_t)(s[8]->nb[1] / 4); }
     a.weights = n->op_params[9];
     if (s[9]) { a.dist_bias = (const float *)s[9]->data; a.n_dist = (int32_t)s[9]->ne[0]; }
-    a.dist_linear = n->op_params[10]; a.out_scale = ext_f(n, 11);
+    a.dist_linear = n->op_params[10]; a.out_scale = ext_f(n, 11); a.softcap = ext_f(n, 12);
     a.gate_per_value = s[8] && s[8]->ne[0] != a.n_head;
 }
 
@@ -189,9 +191,10 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
         }
         case B200_EXT_LATENT_KV_STORE: {
             const int32_t kv_rank = n->op_params[2];
-            B200_CHECK_RC(b200_op_latent_kv_store((const float *)s[0]->data, (int64_t)(s[0]->nb[1] / 4), (const float *)s[1]->data, (const int32_t *)s[2]->data,
-                                                  (const float *)s[3]->data, (const int32_t *)s[4]->data, (float *)s[5]->data, (int64_t)(s[5]->nb[1] / 4), kv_rank,
-                                                  (int32_t)s[0]->ne[0] - kv_rank, n->op_params[5], ext_f(n, 4), ext_f(n, 3), (int32_t)s[0]->ne[1], x.stream));
+            B200_CHECK_RC(b200_op_latent_store((const float *)s[0]->data, (int64_t)(s[0]->nb[1] / 4), (const float *)s[1]->data, (const int32_t *)s[2]->data,
+                                               s[3] ? (const float *)s[3]->data : nullptr, (const int32_t *)s[4]->data, (float *)s[5]->data, (int64_t)(s[5]->nb[1] / 4), kv_rank,
+                                               (int32_t)s[0]->ne[0] - kv_rank, n->op_params[5], ext_f(n, 4), ext_f(n, 3), s[6] ? (float *)s[6]->data : nullptr,
+                                               s[6] ? (int64_t)(s[6]->nb[1] / 4) : 0, s[6] ? (const float *)s[7]->data : nullptr, s[6] ? (int32_t)s[6]->ne[0] : 0, (int32_t)s[0]->ne[1], x.stream));
             break;
         }
         case B200_EXT_LATENT_ATTN: {
@@ -208,6 +211,7 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
             a.kv_rank = n->op_params[2]; a.rot_dim = (int32_t)s[2]->ne[0] - a.kv_rank; a.n_head = (int32_t)s[0]->ne[1]; a.n_tokens = (int32_t)s[0]->ne[2];
             a.n_kv = (int32_t)s[6]->ne[0]; a.window = n->op_params[4]; a.scale = ext_f(n, 3);
             a.bf16_products = n->op_params[5];
+            if (s[8]) { a.gate = (const float *)s[8]->data; a.gate_stride = (int64_t)(s[8]->nb[1] / 4); }
             B200_CHECK_RC(b200_op_latent_attn(&a, x.stream));
             break;
         }
@@ -244,7 +248,7 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
             a.pos = (const int32_t *)s[4]->data; a.freqs = s[5] ? (const float *)s[5]->data : nullptr; a.cells = (const int32_t *)s[6]->data;
             a.k_cache = (float *)s[7]->data; a.k_cache_stride = (int64_t)(s[7]->nb[1] / 4);
             a.v_cache = (float *)s[8]->data; a.v_cache_stride = (int64_t)(s[8]->nb[1] / 4);
-            a.v_unit_rms = n->op_params[9]; a.q_temp_coef = ext_f(n, 10); a.q_temp_every = n->op_params[11];
+            a.v_unit_rms = n->op_params[9]; a.q_temp_coef = ext_f(n, 10); a.q_temp_every = n->op_params[11]; a.rope_mscale = ext_f(n, 12);
             B200_CHECK_RC(b200_op_qkv_store(&a, x.stream));
             break;
         }
@@ -263,7 +267,8 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
             a.q = (const float *)s[0]->data; a.q_stride = (int64_t)(s[0]->nb[1] / 4);
             a.k = (const float *)s[1]->data; a.k_stride = (int64_t)(s[1]->nb[1] / 4);
             a.v = (const float *)s[2]->data; a.v_stride = (int64_t)(s[2]->nb[1] / 4);
-            a.decay = (const float *)s[3]->data;
+            a.decay = s[3] ? (const float *)s[3]->data : nullptr;
+            if (s[8]) { a.z = (const float *)s[8]->data; a.z_stride = (int64_t)(s[8]->nb[1] / 4); a.z_bias = s[9] ? (const float *)s[9]->data : nullptr; a.tau = ext_f(n, 8); }
             a.seq_info = (const int32_t *)s[4]->data; a.n_seq = (int32_t)s[4]->ne[0];
             a.state = (float *)s[5]->data; a.slot_stride = (int64_t)(s[5]->nb[1] / 4);
             a.dst = (float *)n->data; a.dst_stride = (int64_t)(n->nb[1] / 4);
@@ -360,7 +365,7 @@ static void run_ext(ExecCtx &x, const ggml_tensor *n) {
             a.state = (float *)s[8]->data; a.slot_stride = (int64_t)(s[8]->nb[1] / 4);
             a.dst = (float *)n->data; a.dst_stride = (int64_t)(n->nb[1] / 4);
             a.heads = n->op_params[2]; a.kv_heads = n->op_params[3]; a.dim = n->op_params[4]; a.vdim = n->op_params[5]; a.unit_qk = n->op_params[6];
-            a.unit_eps = ext_f(n, 7); a.q_scale = ext_f(n, 8);
+            a.unit_eps = ext_f(n, 7); a.q_scale = ext_f(n, 8); a.channel_decay = s[3]->ne[0] != a.heads;
             B200_CHECK_RC(b200_op_delta_rule_scan(&a, x.stream));
             break;
         }

@@ -79,6 +79,7 @@ __global__ void __launch_bounds__(1024) qkv_store_kernel(const b200_qkv_store_ar
             else if (unit) { u *= sc; w *= sc; }
             float sn, cs;
             sincosf(p * a.freqs[j], &sn, &cs);
+            sn *= a.rope_mscale; cs *= a.rope_mscale;
             const float tq = which ? 1.0f : q_temp;
             dst[e0] = (u * cs - w * sn) * tq;
             dst[e1] = (w * cs + u * sn) * tq;
@@ -109,6 +110,10 @@ __device__ __forceinline__ float sa_dist_bias(const b200_sink_attn_args &a, int 
     if (a.dist_linear) return lin * (float)dist;
     return a.dist_bias ? a.dist_bias[(int64_t)h * a.n_dist + min(dist, a.n_dist - 1)] : 0.f;  // a head's row is contiguous: neighbouring keys share cache lines
 }
+// cap * tanh(s / cap), cap > 0
+__device__ __forceinline__ float sa_cap(float s, float cap) { return cap * tanhf(s / cap); }
+// the same through tanh(x) = 1 - 2 / (1 + e^(2x)) with the fast exponential and division: off by about 2^-23 of the cap at most, whatever s
+__device__ __forceinline__ float sa_cap_fast(float s, float cap, float two_over_cap) { return cap - cap * __fdividef(2.0f, 1.0f + __expf(s * two_over_cap)); }
 __device__ __forceinline__ float sa_sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
 // for weights that are rounded to bf16 right away (8 bits of mantissa): the fast exponential and division are exact enough
 __device__ __forceinline__ float sa_sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
@@ -185,7 +190,12 @@ __global__ void __launch_bounds__(WARPS * 32) sink_attn_kernel(const b200_sink_a
                 for (int i = 0; i < ND; i++) s[u] += q[i] * kv[u][i];
             }
 #pragma unroll
-            for (int u = 0; u < SA_UNROLL; u++) if (vis[u]) s[u] = warp_sum(s[u]) + __shfl_sync(0xffffffffu, my_bias, cu[u] - cb);
+            for (int u = 0; u < SA_UNROLL; u++) {
+                if (!vis[u]) continue;
+                s[u] = warp_sum(s[u]);
+                if (a.softcap > 0.f) s[u] = sa_cap(s[u], a.softcap);
+                s[u] += __shfl_sync(0xffffffffu, my_bias, cu[u] - cb);
+            }
 #pragma unroll
             for (int u = 0; u < SA_UNROLL; u++) {
                 if (!vis[u]) continue;
@@ -388,7 +398,7 @@ __global__ void __launch_bounds__(GM_WARPS * 32) sink_attn_mma_kernel(const b200
     for (int j = 0; j < 2 * VS; j++) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // rows g and g + 8; l: this lane's share of the row sum
     const bool sig = a.weights == B200_ATTN_SIGMOID;
-    const float lin = sa_dist_slope(a, h);
+    const float lin = sa_dist_slope(a, h), two_over_cap = a.softcap > 0.f ? 2.0f / a.softcap : 0.f;
 
     for (int c0 = 0; c0 < a.n_kv; c0 += GM_CELLS) {
         // does any of the warp's tokens see any of the tile's cells?  lane = cell
@@ -426,11 +436,17 @@ __global__ void __launch_bounds__(GM_WARPS * 32) sink_attn_mma_kernel(const b200
 #pragma unroll
         for (int j = 0; j < GM_CELLS / 8; j++) {
 #pragma unroll
+            for (int e = 0; e < 4; e++) s[j][e] *= a.scale;
+            if (a.softcap > 0.f) {
+#pragma unroll
+                for (int e = 0; e < 4; e++) s[j][e] = sa_cap_fast(s[j][e], a.softcap, two_over_cap);
+            }
+#pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int c = j * 8 + 2 * t4 + e;
                 const int xs = cseq[c], xp = cpos[c];
-                s[j][e] = sa_visible(xs, xp, rs0, rp0, a.window, a.keep_first, rl0) ? s[j][e] * a.scale + sa_dist_bias(a, rp0 - xp, h, lin) : -INFINITY;
-                s[j][2 + e] = sa_visible(xs, xp, rs1, rp1, a.window, a.keep_first, rl1) ? s[j][2 + e] * a.scale + sa_dist_bias(a, rp1 - xp, h, lin) : -INFINITY;
+                s[j][e] = sa_visible(xs, xp, rs0, rp0, a.window, a.keep_first, rl0) ? s[j][e] + sa_dist_bias(a, rp0 - xp, h, lin) : -INFINITY;
+                s[j][2 + e] = sa_visible(xs, xp, rs1, rp1, a.window, a.keep_first, rl1) ? s[j][2 + e] + sa_dist_bias(a, rp1 - xp, h, lin) : -INFINITY;
                 mx0 = fmaxf(mx0, s[j][e]); mx1 = fmaxf(mx1, s[j][2 + e]);
             }
         }
@@ -541,21 +557,26 @@ static int launch_sink_attn_mma(const b200_sink_attn_args *a, cudaStream_t st) {
 // The columns of the state never interact: a warp owns LA_CW columns of one (sequence, head) and keeps them in registers over
 // the whole token loop, a lane the rows d = lane, lane + 32, ...  The inputs of LA_CHUNK tokens are staged in shared memory
 // (activation applied once) while the serial loop only does the decayed rank-one update and the column sums.
-constexpr int LA_CW = 4, LA_WARPS = 4, LA_COLS = LA_CW * LA_WARPS, LA_CHUNK = 16, LA_RG = 8;
+// CHAN: every key channel has its own decay per token, sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau), computed once per CTA while the
+// inputs are staged.
+constexpr int LA_CW = 4, LA_WARPS = 4, LA_COLS = LA_CW * LA_WARPS, LA_RG = 8;
+template <int DPL, bool CHAN> constexpr int la_chunk() { return CHAN && DPL > 4 ? 8 : 16; }  // tokens per chunk: a third staged row of 256 values costs registers
 static_assert(LA_RG * LA_CW == 32 && LA_CW == 4, "one partial sum per lane");
 __device__ __forceinline__ float la_act(float x, int act) { return act ? x / (1.0f + expf(-x)) : x; }
-template <int DPL>
+__device__ __forceinline__ float la_channel_decay(float z, float inv_tau) { return expf(-inv_tau * (fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z))))); }
+template <int DPL, bool CHAN>
 __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b200_linear_attn_args a) {
-    extern __shared__ float sm_[];  // q [LA_CHUNK][32 DPL], k [LA_CHUNK][32 DPL], v [LA_CHUNK][LA_COLS]
+    constexpr int LA_CHUNK = la_chunk<DPL, CHAN>();
+    extern __shared__ float sm_[];  // q [LA_CHUNK][32 DPL], k [LA_CHUNK][32 DPL], v [LA_CHUNK][LA_COLS], with CHAN decays [LA_CHUNK][32 DPL]
     const int h = blockIdx.y, s = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
     const int D = a.dim, V = a.vdim;
     const int first = a.seq_info[s], count = a.seq_info[a.n_seq + s], slot = a.seq_info[2 * a.n_seq + s], fresh = a.seq_info[3 * a.n_seq + s];
     if (count <= 0) return;
     const int cb = blockIdx.x * LA_COLS, col0 = cb + warp * LA_CW;
-    float *sq = sm_, *sk = sq + LA_CHUNK * 32 * DPL, *sv = sk + LA_CHUNK * 32 * DPL;  // rows padded to 32 DPL values
+    float *sq = sm_, *sk = sq + LA_CHUNK * 32 * DPL, *sv = sk + LA_CHUNK * 32 * DPL, *sw = sv + LA_CHUNK * LA_COLS;  // rows padded to 32 DPL values
     float *Sp = a.state + (int64_t)slot * a.slot_stride + ((int64_t)h * V + col0) * D;
-    const float decay = a.decay[h];
+    const float decay = CHAN ? 0.f : a.decay[h], inv_tau = CHAN ? 1.0f / a.tau : 0.f;
     float S[LA_CW][DPL];
 #pragma unroll
     for (int i = 0; i < DPL; i++) {
@@ -566,7 +587,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
     // the inputs of the next chunk travel to registers while the current chunk is worked on: a chunk costs one trip to L2 / HBM that
     // overlaps the serial loop instead of standing in front of it
     constexpr int DP = 32 * DPL, NQ = LA_CHUNK * DP / (LA_WARPS * 32), NVV = LA_CHUNK * LA_COLS / (LA_WARPS * 32);
-    float pq[NQ], pk[NQ], pv[NVV];
+    float pq[NQ], pk[NQ], pv[NVV], pz[CHAN ? NQ : 1];
     auto fetch = [&](int t0) {
         const int nt = min(LA_CHUNK, count - t0);
 #pragma unroll
@@ -576,6 +597,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
             const int64_t tok = first + t0 + tt;
             pq[j] = ok ? a.q[tok * a.q_stride + (int64_t)h * D + d] : 0.f;
             pk[j] = ok ? a.k[tok * a.k_stride + (int64_t)h * D + d] : 0.f;
+            if (CHAN) pz[CHAN ? j : 0] = ok ? a.z[tok * a.z_stride + (int64_t)h * D + d] + (a.z_bias ? a.z_bias[h * D + d] : 0.f) : 0.f;
         }
 #pragma unroll
         for (int j = 0; j < NVV; j++) {
@@ -591,6 +613,10 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
         for (int j = 0; j < NQ; j++) { sq[tid + j * LA_WARPS * 32] = la_act(pq[j], a.act); sk[tid + j * LA_WARPS * 32] = la_act(pk[j], a.act) * a.k_scale; }
 #pragma unroll
         for (int j = 0; j < NVV; j++) sv[tid + j * LA_WARPS * 32] = la_act(pv[j], a.act);
+        if (CHAN) {
+#pragma unroll
+            for (int j = 0; j < NQ; j++) sw[tid + j * LA_WARPS * 32] = la_channel_decay(pz[CHAN ? j : 0], inv_tau);
+        }
         __syncthreads();
         if (a.n_dims > 0) {  // rotation of entry i with entry i + n_dims / 2 where the rows wait (the scale on k commutes with it)
             const int half = a.n_dims / 2;
@@ -614,15 +640,15 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
             for (int u = 0; u < LA_RG; u++) {
                 const int tt = tt0 + u;
                 if (tt < nt) {  // warp-uniform
-                    float qv[DPL], kv[DPL];
+                    float qv[DPL], kv[DPL], wv[DPL];
 #pragma unroll
-                    for (int i = 0; i < DPL; i++) { const int d = lane + 32 * i; qv[i] = sq[tt * DP + d]; kv[i] = sk[tt * DP + d]; }
+                    for (int i = 0; i < DPL; i++) { const int d = lane + 32 * i; qv[i] = sq[tt * DP + d]; kv[i] = sk[tt * DP + d]; wv[i] = CHAN ? sw[tt * DP + d] : decay; }
 #pragma unroll
                     for (int c = 0; c < LA_CW; c++) {
                         const float vc = sv[tt * LA_COLS + warp * LA_CW + c];
                         float acc = 0.f;
 #pragma unroll
-                        for (int i = 0; i < DPL; i++) { S[c][i] = decay * S[c][i] + kv[i] * vc; acc += S[c][i] * qv[i]; }
+                        for (int i = 0; i < DPL; i++) { S[c][i] = wv[i] * S[c][i] + kv[i] * vc; acc += S[c][i] * qv[i]; }
                         part[u * LA_CW + c] = acc;
                     }
                 } else {
@@ -651,21 +677,27 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
     }
 }
 
-template <int DPL>
-static int launch_linear_attn(const b200_linear_attn_args *a, cudaStream_t st) {
+template <int DPL, bool CHAN>
+static int launch_linear_attn2(const b200_linear_attn_args *a, cudaStream_t st) {
     const dim3 grid((unsigned)((a->vdim + LA_COLS - 1) / LA_COLS), (unsigned)a->heads, (unsigned)a->n_seq);
-    const size_t smem = (size_t)LA_CHUNK * (2 * 32 * DPL + LA_COLS) * 4;
-    linear_attn_scan_kernel<DPL><<<grid, LA_WARPS * 32, smem, st>>>(*a);
+    const size_t smem = (size_t)la_chunk<DPL, CHAN>() * ((CHAN ? 3 : 2) * 32 * DPL + LA_COLS) * 4;
+    linear_attn_scan_kernel<DPL, CHAN><<<grid, LA_WARPS * 32, smem, st>>>(*a);
     B200_CUDA_TRY(cudaGetLastError());
     return B200_OK;
 }
+template <int DPL>
+static int launch_linear_attn(const b200_linear_attn_args *a, cudaStream_t st) { return a->z ? launch_linear_attn2<DPL, true>(a, st) : launch_linear_attn2<DPL, false>(a, st); }
 
 }  // namespace b200
 
 using namespace b200;
 
-extern "C" int b200_op_qkv_store(const b200_qkv_store_args *a, b200_stream_t stream) {
-    OPX_REQUIRE(a && a->q && a->k && a->v && a->pos && a->cells && a->k_cache && a->v_cache && (a->freqs || a->n_dims == 0), B200_ERR_INVALID, "b200_op_qkv_store: NULL argument");
+extern "C" int b200_op_qkv_store(const b200_qkv_store_args *args, b200_stream_t stream) {
+    OPX_REQUIRE(args, B200_ERR_INVALID, "b200_op_qkv_store: NULL argument");
+    b200_qkv_store_args copy = *args;
+    if (copy.rope_mscale == 0.0f) copy.rope_mscale = 1.0f;
+    const b200_qkv_store_args *a = &copy;
+    OPX_REQUIRE(a->q && a->k && a->v && a->pos && a->cells && a->k_cache && a->v_cache && (a->freqs || a->n_dims == 0), B200_ERR_INVALID, "b200_op_qkv_store: NULL argument");
     OPX_REQUIRE(a->n_head > 0 && a->n_head_kv > 0 && a->n_head % a->n_head_kv == 0 && a->dim > 0 && a->vdim > 0 && a->n_dims >= 0 && a->n_dims % 2 == 0 && a->n_dims <= a->dim &&
                 a->n_tokens >= 0 && a->k_cache_stride >= (int64_t)a->n_head_kv * a->dim && a->v_cache_stride >= (int64_t)a->n_head_kv * a->vdim, B200_ERR_INVALID,
                 "b200_op_qkv_store: bad sizes");
@@ -697,6 +729,7 @@ extern "C" int b200_op_sink_attn_ws(const b200_sink_attn_args *args, void *works
     OPX_REQUIRE(a->n_head > 0 && a->n_head <= 65535 && a->n_head_kv > 0 && a->n_head % a->n_head_kv == 0 && a->dim > 0 && a->dim <= 256 && a->vdim > 0 && a->vdim <= 256 &&
                 a->n_tokens >= 0 && a->n_kv >= 0 && a->window >= 0 && a->keep_first >= 0 && a->chunk >= 0, B200_ERR_UNSUPPORTED, "b200_op_sink_attn: head sizes up to 256, heads up to 65535");
     OPX_REQUIRE((a->weights == B200_ATTN_SOFTMAX || a->weights == B200_ATTN_SIGMOID) && (!a->dist_bias || a->n_dist > 0), B200_ERR_INVALID, "b200_op_sink_attn: weight kind / distance table");
+    OPX_REQUIRE(a->softcap >= 0.f, B200_ERR_INVALID, "b200_op_sink_attn: soft cap below zero");
     if (a->n_tokens == 0) return B200_OK;
     const cudaStream_t st = (cudaStream_t)stream;
     if (sink_attn_mma_ok(a)) return launch_sink_attn_mma(a, st);
@@ -716,7 +749,8 @@ extern "C" int b200_op_linear_attn_scan(const b200_linear_attn_args *args, b200_
     if (copy.k_scale == 0.0f) copy.k_scale = 1.0f;
     const b200_linear_attn_args *a = &copy;
     OPX_REQUIRE(a->n_dims == 0 || (a->n_dims > 0 && a->n_dims % 2 == 0 && a->n_dims <= a->dim && a->pos && a->freqs), B200_ERR_INVALID, "b200_op_linear_attn_scan: rotation does not fit dim");
-    OPX_REQUIRE(a->q && a->k && a->v && a->decay && a->seq_info && a->state && a->dst, B200_ERR_INVALID, "b200_op_linear_attn_scan: NULL argument");
+    OPX_REQUIRE(a->q && a->k && a->v && (a->decay || a->z) && a->seq_info && a->state && a->dst, B200_ERR_INVALID, "b200_op_linear_attn_scan: NULL argument");
+    OPX_REQUIRE(!a->z || a->tau > 0.f, B200_ERR_INVALID, "b200_op_linear_attn_scan: tau must be positive");
     OPX_REQUIRE(a->heads > 0 && a->heads <= 65535 && a->dim > 0 && a->dim <= 256 && a->vdim > 0 && a->n_seq >= 0 && a->n_seq <= 65535 &&
                 a->slot_stride >= (int64_t)a->heads * a->dim * a->vdim, B200_ERR_UNSUPPORTED, "b200_op_linear_attn_scan: dim up to 256");
     if (a->n_seq == 0) return B200_OK;

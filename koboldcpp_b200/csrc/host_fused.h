@@ -65,10 +65,20 @@ inline int place_into(b200_llama *m, const std::string &fused, const char *part_
 }
 
 // per-pair rotation frequencies base^(-2i/dims), in double, rounded once; BANDS rescales by wavelength: short ones are kept, long
-// ones divided by the factor, the band between blended linearly in original / wavelength
-inline void rope_freqs(const b200_layer_params &lp, std::vector<float> &f) {
+// ones divided by the factor, the band between blended linearly in original / wavelength; YARN blends the kept and the divided frequency
+// linearly in the pair's index between the pairs that turn yarn_fast and yarn_slow times within the original length, and its factor on
+// sine and cosine goes to *mscale (1 without it)
+inline void rope_freqs(const b200_layer_params &lp, std::vector<float> &f, float *mscale = nullptr) {
     const int dims = lp.rope_dims;
     f.resize((size_t)(dims / 2));
+    const bool yarn = lp.rope_scaling == B200_ROPE_SCALING_YARN;
+    double lo = 0.0, hi = 0.0;
+    if (yarn) {
+        auto pair_of = [&](double turns) { return dims * log((double)lp.yarn_original / (2.0 * M_PI * turns)) / (2.0 * log((double)lp.rope_base)); };
+        lo = fmax(floor(pair_of(lp.yarn_fast)), 0.0);
+        hi = fmin(ceil(pair_of(lp.yarn_slow)), (double)dims - 1.0);
+    }
+    if (mscale) *mscale = yarn ? (float)(0.1 * log((double)lp.yarn_factor) + 1.0) : 1.0f;
     for (int i = 0; i < dims / 2; i++) {
         double fi = pow((double)lp.rope_base, -2.0 * i / dims);
         if (lp.rope_scaling == B200_ROPE_SCALING_BANDS) {
@@ -78,6 +88,10 @@ inline void rope_freqs(const b200_layer_params &lp, std::vector<float> &f) {
                 const double s = (orig / wl - lp.band_low) / ((double)lp.band_high - lp.band_low);
                 fi = (1.0 - s) * fi / lp.yarn_factor + s * fi;
             }
+        }
+        if (yarn) {
+            const double ramp = fmin(fmax((i - lo) / fmax(hi - lo, 0.001), 0.0), 1.0);
+            fi = fi / lp.yarn_factor * ramp + fi * (1.0 - ramp);
         }
         f[(size_t)i] = (float)fi;
     }

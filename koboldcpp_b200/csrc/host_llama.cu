@@ -8,7 +8,7 @@
 
 const Arch *b200::host::find_arch(int32_t id) {
     return id == B200_ARCH_GENESUN ? genesun_arch() : id == B200_ARCH_GALIRAX ? galirax_arch() : id == B200_ARCH_ZEVOPEL ? zevopel_arch() : id == B200_ARCH_MEDODRA ? medodra_arch() :
-           id == B200_ARCH_MAFUZEN ? mafuzen_arch() : nullptr;
+           id == B200_ARCH_MAFUZEN ? mafuzen_arch() : id == B200_ARCH_TUGEZEN ? tugezen_arch() : nullptr;
 }
 
 extern "C" int b200_llama_new(const b200_llama_params *p, b200_llama **out) {

@@ -265,6 +265,7 @@ const Arch *galirax_arch();
 const Arch *zevopel_arch();
 const Arch *medodra_arch();
 const Arch *mafuzen_arch();
+const Arch *tugezen_arch();
 
 }  // namespace host
 }  // namespace b200

@@ -11,11 +11,23 @@
 namespace b200 {
 using namespace opx;
 
+// the sigmoid gate of a head's result (1 without one)
+__device__ __forceinline__ float la_head_gate(const b200_latent_attn_args &a, int64_t t, int h) { return a.gate ? 1.0f / (1.0f + expf(-a.gate[t * a.gate_stride + h])) : 1.0f; }
+
 __global__ void latent_kv_store_kernel(const float *__restrict__ dkv, int64_t dkv_stride, const float *__restrict__ w, const int32_t *__restrict__ pos,
                                        const float *__restrict__ freqs, const int32_t *__restrict__ cells, float *__restrict__ cache, int64_t cache_stride,
-                                       int kv_rank, int rot_dim, int n_dims, float mscale, float eps) {
+                                       int kv_rank, int rot_dim, int n_dims, float mscale, float eps, float *__restrict__ q, int64_t q_stride,
+                                       const float *__restrict__ q_w, int q_rank) {
     __shared__ float sh[32];
     const int t = blockIdx.x;
+    if (blockIdx.y == 1) {  // the token's query latent, normed where it lies
+        float *y = q + (int64_t)t * q_stride, ss = 0.f;
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) ss += y[i] * y[i];
+        ss = block_sum(ss, sh);
+        const float f = 1.0f / sqrtf(ss / (float)q_rank + eps);
+        for (int i = threadIdx.x; i < q_rank; i += blockDim.x) y[i] = y[i] * f * q_w[i];
+        return;
+    }
     const float *x = dkv + (int64_t)t * dkv_stride;
     float *row = cache + (int64_t)cells[t] * cache_stride;
     float s = 0.f;
@@ -26,7 +38,7 @@ __global__ void latent_kv_store_kernel(const float *__restrict__ dkv, int64_t dk
     const float *xr = x + kv_rank;
     float *rr = row + kv_rank;
     const int half = n_dims / 2;
-    const float p = (float)pos[t];
+    const float p = n_dims > 0 ? (float)pos[t] : 0.f;
     for (int j = threadIdx.x; j < half + (rot_dim - n_dims); j += blockDim.x) {
         if (j >= half) { rr[n_dims + j - half] = xr[n_dims + j - half]; continue; }
         float sn, cs;
@@ -125,7 +137,7 @@ __global__ void __launch_bounds__(WARPS * 32) latent_attn_kernel(const b200_late
     __syncthreads();
     if (threadIdx.x < WARPS) sl[threadIdx.x] = sm[threadIdx.x] == -INFINITY ? 0.f : expf(sm[threadIdx.x] - M);  // the warp's weight in the merge
     __syncthreads();
-    const float inv = 1.0f / L;
+    const float inv = (L > 0.f ? 1.0f / L : 0.f) * la_head_gate(a, t, h);
     float *out = a.dst + (int64_t)h * a.dst_s_head + (int64_t)t * a.dst_s_tok;
     for (int j = threadIdx.x; j < KR; j += blockDim.x) {
         float o = 0.f;
@@ -194,7 +206,8 @@ __global__ void __launch_bounds__(LT_HEADS * 32) latent_attn_tile_kernel(const b
     const float sink = a.sink ? a.sink[h] : -INFINITY;
     const float M = fmaxf(m, sink);
     const float f = m == -INFINITY ? 0.f : expf(m - M);
-    const float inv = 1.0f / (l * f + (a.sink ? expf(sink - M) : 0.f));
+    const float den = l * f + (a.sink ? expf(sink - M) : 0.f);
+    const float inv = (den > 0.f ? 1.0f / den : 0.f) * la_head_gate(a, t, h);
     float *out = a.dst + (int64_t)h * a.dst_s_head + (int64_t)t * a.dst_s_tok;
 #pragma unroll
     for (int i = 0; i < NL; i++) { const int j = lane + 32 * i; if (j < KR) out[j] = acc[i] * f * inv; }
@@ -429,7 +442,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32, NI <= 5 ? 2 : 1) latent_attn_mm
         const float M = fmaxf(m_row, sink);
         const float f = m_row == -INFINITY ? 0.f : expf(m_row - M);
         const float den = l_row * f + (a.sink ? expf(sink - M) : 0.f);
-        alph[my_r] = den > 0.f ? f / den : 0.f;
+        alph[my_r] = (den > 0.f ? f / den : 0.f) * (t0 + my_r < a.n_tokens ? la_head_gate(a, t0 + my_r, h) : 1.0f);
     }
     __syncthreads();
     const float w[2] = {alph[g], alph[g + 8]};
@@ -508,17 +521,22 @@ static int launch_latent_attn(const b200_latent_attn_args *a, cudaStream_t st) {
 
 using namespace b200;
 
-extern "C" int b200_op_latent_kv_store(const float *dkv, int64_t dkv_stride, const float *w, const int32_t *pos, const float *freqs, const int32_t *cells,
-                                       float *cache, int64_t cache_stride, int32_t kv_rank, int32_t rot_dim, int32_t n_dims, float mscale, float eps,
-                                       int32_t n_tokens, b200_stream_t stream) {
-    OPX_REQUIRE(dkv && w && pos && freqs && cells && cache, B200_ERR_INVALID, "b200_op_latent_kv_store: NULL argument");
+extern "C" int b200_op_latent_store(const float *dkv, int64_t dkv_stride, const float *w, const int32_t *pos, const float *freqs, const int32_t *cells,
+                                    float *cache, int64_t cache_stride, int32_t kv_rank, int32_t rot_dim, int32_t n_dims, float mscale, float eps,
+                                    float *q, int64_t q_stride, const float *q_w, int32_t q_rank, int32_t n_tokens, b200_stream_t stream) {
+    OPX_REQUIRE(dkv && w && cells && cache && (n_dims == 0 || (pos && freqs)) && (!q || (q_w && q_rank > 0 && q_stride >= q_rank)), B200_ERR_INVALID, "b200_op_latent_kv_store: NULL argument");
     OPX_REQUIRE(kv_rank > 0 && rot_dim >= 0 && n_dims >= 0 && n_dims % 2 == 0 && n_dims <= rot_dim && cache_stride >= kv_rank + rot_dim && n_tokens >= 0,
                 B200_ERR_INVALID, "b200_op_latent_kv_store: bad sizes");
     if (n_tokens == 0) return B200_OK;
-    latent_kv_store_kernel<<<(unsigned)n_tokens, 128, 0, (cudaStream_t)stream>>>(dkv, dkv_stride, w, pos, freqs, cells, cache, cache_stride, kv_rank, rot_dim,
-                                                                                 n_dims, mscale, eps);
+    latent_kv_store_kernel<<<dim3((unsigned)n_tokens, q ? 2 : 1), n_tokens <= 64 ? 512 : 128, 0, (cudaStream_t)stream>>>(dkv, dkv_stride, w, pos, freqs, cells, cache, cache_stride, kv_rank, rot_dim,
+                                                                                                                       n_dims, mscale, eps, q, q_stride, q_w, q_rank);
     B200_CUDA_TRY(cudaGetLastError());
     return B200_OK;
+}
+extern "C" int b200_op_latent_kv_store(const float *dkv, int64_t dkv_stride, const float *w, const int32_t *pos, const float *freqs, const int32_t *cells,
+                                       float *cache, int64_t cache_stride, int32_t kv_rank, int32_t rot_dim, int32_t n_dims, float mscale, float eps,
+                                       int32_t n_tokens, b200_stream_t stream) {
+    return b200_op_latent_store(dkv, dkv_stride, w, pos, freqs, cells, cache, cache_stride, kv_rank, rot_dim, n_dims, mscale, eps, nullptr, 0, nullptr, 0, n_tokens, stream);
 }
 
 extern "C" int b200_op_latent_attn(const b200_latent_attn_args *a, b200_stream_t stream) {

@@ -355,8 +355,8 @@ __global__ void __launch_bounds__(1024) norm_chain_kernel(const b200_norm_chain_
             for (int k = 0; k < VPT; k++) v[k] += u[k];
         }
     }
-    float mean, scale;
-    row_statistics(v, ok, a.kind1 == B200_NORM_LAYER, cnt, n, a.eps, sh[0], mean, scale);
+    float mean = 0.f, scale = 1.0f;
+    if (a.kind1 != B200_NORM_NONE) row_statistics(v, ok, a.kind1 == B200_NORM_LAYER, cnt, n, a.eps, sh[0], mean, scale);
 #pragma unroll
     for (int k = 0; k < VPT; k++) v[k] = ok[k] ? rv[k] + ((v[k] - mean) * scale * w1[k] + b1[k]) : 0.f;
     store(a.x + t * a.x_stride, v);
@@ -408,7 +408,7 @@ extern "C" int b200_op_norm_chain(const b200_norm_chain_args *args, b200_stream_
     b200_norm_chain_args a = *args;
     if (a.y_scale == 0.0f) a.y_scale = 1.0f;
     OPX_REQUIRE(a.n >= 0 && a.n <= 16384 && a.n_y >= 1 && a.n_tok >= 0, B200_ERR_UNSUPPORTED, "b200_op_norm_chain: rows of at most 16384 values, at least one result per token");
-    OPX_REQUIRE((a.kind1 == B200_NORM_LAYER || a.kind1 == B200_NORM_RMS) && (!a.h || a.kind2 == B200_NORM_LAYER || a.kind2 == B200_NORM_RMS), B200_ERR_INVALID, "b200_op_norm_chain: norm kind");
+    OPX_REQUIRE((a.kind1 == B200_NORM_LAYER || a.kind1 == B200_NORM_RMS || a.kind1 == B200_NORM_NONE) && (!a.h || a.kind2 == B200_NORM_LAYER || a.kind2 == B200_NORM_RMS), B200_ERR_INVALID, "b200_op_norm_chain: norm kind");
     if (a.n == 0 || a.n_tok == 0) return B200_OK;
     const int n = (int)a.n;
     const int rb = n <= 256 ? 64 : n <= 512 ? 128 : n <= 1024 ? 256 : n <= 2048 ? 512 : 1024, vpt = (n + rb - 1) / rb;

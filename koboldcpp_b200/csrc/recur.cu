@@ -67,13 +67,16 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const b200_short_conv_a
 // 4 (r + 8 i) .. + 3 of each in registers over the whole token loop, so a sum over a column is three exchanges among 8 lanes and
 // the q and k values a lane reads from shared memory serve DR_CPL columns (the loads, not the arithmetic, are what two CTAs on one
 // SM compete for).
-// The inputs of DR_CHUNK tokens are staged in shared memory: q and k as unit vectors (q scaled), q.k, the decay and beta once per
+// The inputs of DR_CHUNK tokens (16, or 8) are staged in shared memory: q and k as unit vectors (q scaled), q.k, the decay and beta once per
 // token; the next chunk's values travel to registers while the current chunk is worked on.
-constexpr int DR_CW = 4, DR_CPL = 1, DR_WARPS = 8, DR_COLS = DR_CW * DR_CPL * DR_WARPS, DR_CHUNK = 16, DR_TPW = DR_CHUNK / DR_WARPS;
-template <int DQ>  // float4 groups per lane: dim <= 32 DQ
+// CHAN: the decay is one factor per key channel (row of S) instead of one per head.  The old column is multiplied by it first, then
+// ks, qs are sums over the decayed column and  o_j = qs + (q.k) u_j;  the factors of a chunk are staged like q and k.
+constexpr int DR_CW = 4, DR_CPL = 1, DR_WARPS = 8, DR_COLS = DR_CW * DR_CPL * DR_WARPS;
+template <int DQ, bool CHAN>  // float4 groups per lane: dim <= 32 DQ
 __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b200_delta_rule_args a) {
-    constexpr int DP = 32 * DQ;
+    constexpr int DP = 32 * DQ, DR_CHUNK = CHAN && DQ > 4 ? 8 : 16, DR_TPW = DR_CHUNK / DR_WARPS;  // (three staged rows of 256 values: half the tokens fit)
     __shared__ __align__(16) float sq[DR_CHUNK][DP], sk[DR_CHUNK][DP];
+    __shared__ __align__(16) float sgc[CHAN ? DR_CHUNK : 1][CHAN ? DP : 4];
     __shared__ float sv[DR_CHUNK][DR_COLS], sqk[DR_CHUNK], sg[DR_CHUNK], sbeta[DR_CHUNK];
     const int h = blockIdx.y, s = blockIdx.z, kvh = h / (a.heads / a.kv_heads);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
@@ -92,11 +95,11 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
                 const int d = 4 * (r + 8 * i) + e;
                 S[c][i][e] = (!fresh && d < D && cb + lc0 + DR_CW * c < V) ? Sp[(int64_t)DR_CW * c * D + d] : 0.f;
             }
-    const float decay_rate = expf(a.a_log[h]), dtb = a.dt_bias ? a.dt_bias[h] : 0.f;
+    const float decay_rate = expf(a.a_log[h]), dtb = !CHAN && a.dt_bias ? a.dt_bias[h] : 0.f;
     // staging: the raw values of a chunk travel to registers (every thread a slice of the chunk), are parked in shared memory, and
     // warp w then turns the tokens w, w + DR_WARPS, ... into unit vectors in place
     constexpr int NQ = DR_CHUNK * DP / (DR_WARPS * 32), NVV = (DR_CHUNK * DR_COLS) / (DR_WARPS * 32);
-    float pq[NQ], pk[NQ], pv[NVV], pa = 0.f, pb = 0.f;
+    float pq[NQ], pk[NQ], pg[CHAN ? NQ : 1], pv[NVV], pa = 0.f, pb = 0.f;
     auto fetch = [&](int t0) {
         const int nt = min(DR_CHUNK, count - t0);
 #pragma unroll
@@ -106,6 +109,7 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
             const int64_t tok = first + t0 + tt;
             pq[j] = ok ? a.q[tok * a.q_stride + (int64_t)kvh * D + d] : 0.f;
             pk[j] = ok ? a.k[tok * a.k_stride + (int64_t)kvh * D + d] : 0.f;
+            if (CHAN) pg[CHAN ? j : 0] = ok ? a.a[tok * a.a_stride + (int64_t)h * D + d] + (a.dt_bias ? a.dt_bias[(int64_t)h * D + d] : 0.f) : 0.f;
         }
 #pragma unroll
         for (int j = 0; j < NVV; j++) {
@@ -113,7 +117,7 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
             pv[j] = (tt < nt && cb + c < V) ? a.v[(int64_t)(first + t0 + tt) * a.v_stride + (int64_t)h * V + cb + c] : 0.f;
         }
         if (tid < DR_CHUNK) {
-            pa = tid < nt ? a.a[(int64_t)(first + t0 + tid) * a.a_stride + h] : 0.f;
+            if (!CHAN) pa = tid < nt ? a.a[(int64_t)(first + t0 + tid) * a.a_stride + h] : 0.f;
             pb = tid < nt ? a.b[(int64_t)(first + t0 + tid) * a.b_stride + h] : 0.f;
         }
     };
@@ -125,8 +129,12 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
         for (int j = 0; j < NQ; j++) { (&sq[0][0])[tid + j * DR_WARPS * 32] = pq[j]; (&sk[0][0])[tid + j * DR_WARPS * 32] = pk[j]; }
 #pragma unroll
         for (int j = 0; j < NVV; j++) (&sv[0][0])[tid + j * DR_WARPS * 32] = pv[j];
+        if (CHAN) {
+#pragma unroll
+            for (int j = 0; j < NQ; j++) (&sgc[0][0])[tid + j * DR_WARPS * 32] = expf(-decay_rate * softplus_f(pg[CHAN ? j : 0]));
+        }
         if (tid < DR_CHUNK) {
-            sg[tid] = expf(-decay_rate * softplus_f(pa + dtb));
+            if (!CHAN) sg[tid] = expf(-decay_rate * softplus_f(pa + dtb));
             sbeta[tid] = sigmoidf_(pb);
         }
         __syncthreads();
@@ -163,6 +171,11 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
             for (int i = 0; i < DQ; i++) {
                 kv[i] = *reinterpret_cast<const float4 *>(&sk[tt][4 * (r + 8 * i)]);
                 const float4 qv = *reinterpret_cast<const float4 *>(&sq[tt][4 * (r + 8 * i)]);
+                if (CHAN) {
+                    const float4 gv = *reinterpret_cast<const float4 *>(&sgc[CHAN ? tt : 0][CHAN ? 4 * (r + 8 * i) : 0]);
+#pragma unroll
+                    for (int c = 0; c < DR_CPL; c++) { S[c][i][0] *= gv.x; S[c][i][1] *= gv.y; S[c][i][2] *= gv.z; S[c][i][3] *= gv.w; }
+                }
 #pragma unroll
                 for (int c = 0; c < DR_CPL; c++) {
                     ks[c] += (kv[i].x * S[c][i][0] + kv[i].z * S[c][i][2]) + (kv[i].y * S[c][i][1] + kv[i].w * S[c][i][3]);
@@ -173,7 +186,7 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
             for (int off = 4; off >= 1; off >>= 1)
 #pragma unroll
                 for (int c = 0; c < DR_CPL; c++) { ks[c] += __shfl_xor_sync(0xffffffffu, ks[c], off); qs[c] += __shfl_xor_sync(0xffffffffu, qs[c], off); }
-            const float g = sg[tt];
+            const float g = CHAN ? 1.0f : sg[tt];
 #pragma unroll
             for (int c = 0; c < DR_CPL; c++) {
                 const float u = sbeta[tt] * (sv[tt][lc0 + DR_CW * c] - g * ks[c]);
@@ -197,13 +210,16 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
             }
 }
 
-template <int DQ>
-static int launch_delta_rule(const b200_delta_rule_args *a, cudaStream_t st) {
+template <int DQ, bool CHAN>
+static int launch_delta_rule2(const b200_delta_rule_args *a, cudaStream_t st) {
     const dim3 grid((unsigned)((a->vdim + DR_COLS - 1) / DR_COLS), (unsigned)a->heads, (unsigned)a->n_seq);
-    delta_rule_scan_kernel<DQ><<<grid, DR_WARPS * 32, 0, st>>>(*a);
+    delta_rule_scan_kernel<DQ, CHAN><<<grid, DR_WARPS * 32, 0, st>>>(*a);
     B200_CUDA_TRY(cudaGetLastError());
     return B200_OK;
 }
+
+template <int DQ>
+static int launch_delta_rule(const b200_delta_rule_args *a, cudaStream_t st) { return a->channel_decay ? launch_delta_rule2<DQ, true>(a, st) : launch_delta_rule2<DQ, false>(a, st); }
 
 // ------------------------------------------------------------------------------------------------ minGRU
 // S_t = (1 - z_t) S_(t-1) + z_t c_t is linear in S, so a stretch of tokens acts on the state as S -> A S + B.  A CTA takes 32

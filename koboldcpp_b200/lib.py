@@ -70,7 +70,7 @@ class LatentAttnArgs(C.Structure):
                 ("q_rot_s_tok", C.c_int64), ("cache", C.c_void_p), ("cache_stride", C.c_int64), ("cell_seq", C.c_void_p), ("cell_pos", C.c_void_p),
                 ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p), ("sink", C.c_void_p), ("dst", C.c_void_p), ("dst_s_head", C.c_int64), ("dst_s_tok", C.c_int64),
                 ("kv_rank", C.c_int32), ("rot_dim", C.c_int32), ("n_head", C.c_int32), ("n_tokens", C.c_int32), ("n_kv", C.c_int32), ("window", C.c_int32),
-                ("scale", C.c_float), ("bf16_products", C.c_int32)]
+                ("scale", C.c_float), ("bf16_products", C.c_int32), ("gate", C.c_void_p), ("gate_stride", C.c_int64)]
 
 
 class MlstmArgs(C.Structure):
@@ -88,7 +88,8 @@ class QkvStoreArgs(C.Structure):
                 ("pos", C.c_void_p), ("cells", C.c_void_p), ("freqs", C.c_void_p), ("k_cache", C.c_void_p), ("k_cache_stride", C.c_int64),
                 ("v_cache", C.c_void_p), ("v_cache_stride", C.c_int64), ("n_head", C.c_int32), ("n_head_kv", C.c_int32), ("dim", C.c_int32),
                 ("vdim", C.c_int32), ("n_dims", C.c_int32), ("n_tokens", C.c_int32), ("eps", C.c_float), ("norm_per_head", C.c_int32), ("rope_halves", C.c_int32),
-                ("v_unit_rms", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32), ("qk_unit_rms", C.c_int32)]
+                ("v_unit_rms", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32), ("qk_unit_rms", C.c_int32),
+                ("rope_mscale", C.c_float)]
 
 
 class SinkAttnArgs(C.Structure):
@@ -99,7 +100,7 @@ class SinkAttnArgs(C.Structure):
                 ("vdim", C.c_int32), ("n_tokens", C.c_int32), ("n_kv", C.c_int32), ("window", C.c_int32), ("keep_first", C.c_int32), ("scale", C.c_float),
                 ("bf16_products", C.c_int32), ("chunk", C.c_int32), ("gate", C.c_void_p), ("gate_stride", C.c_int64),
                 ("weights", C.c_int32), ("dist_bias", C.c_void_p), ("n_dist", C.c_int32), ("dist_linear", C.c_int32), ("gate_per_value", C.c_int32),
-                ("out_scale", C.c_float)]
+                ("out_scale", C.c_float), ("softcap", C.c_float)]
 
 
 class LinearAttnArgs(C.Structure):
@@ -107,7 +108,7 @@ class LinearAttnArgs(C.Structure):
     _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("q_stride", C.c_int64), ("k_stride", C.c_int64), ("v_stride", C.c_int64),
                 ("decay", C.c_void_p), ("seq_info", C.c_void_p), ("n_seq", C.c_int32), ("state", C.c_void_p), ("slot_stride", C.c_int64),
                 ("dst", C.c_void_p), ("dst_stride", C.c_int64), ("heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("act", C.c_int32), ("k_scale", C.c_float),
-                ("pos", C.c_void_p), ("freqs", C.c_void_p), ("n_dims", C.c_int32)]
+                ("pos", C.c_void_p), ("freqs", C.c_void_p), ("n_dims", C.c_int32), ("z", C.c_void_p), ("z_stride", C.c_int64), ("z_bias", C.c_void_p), ("tau", C.c_float)]
 
 
 class ShortConvArgs(C.Structure):
@@ -123,7 +124,7 @@ class DeltaRuleArgs(C.Structure):
                 ("a", C.c_void_p), ("b", C.c_void_p), ("a_stride", C.c_int64), ("b_stride", C.c_int64), ("a_log", C.c_void_p), ("dt_bias", C.c_void_p),
                 ("seq_info", C.c_void_p), ("n_seq", C.c_int32), ("state", C.c_void_p), ("slot_stride", C.c_int64), ("dst", C.c_void_p), ("dst_stride", C.c_int64),
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("unit_qk", C.c_int32), ("unit_eps", C.c_float),
-                ("q_scale", C.c_float)]
+                ("q_scale", C.c_float), ("channel_decay", C.c_int32)]
 
 
 class MinGruArgs(C.Structure):

@@ -20,7 +20,7 @@ class LlamaParams(C.Structure):
                 ("rms_eps", C.c_float), ("rope_freq_base", C.c_float), ("rope_freq_scale", C.c_float),
                 ("main_device", C.c_int32), ("n_split_devices", C.c_int32), ("tensor_split", C.c_float * 16),
                 ("tp_rank", C.c_int32), ("tp_world", C.c_int32), ("arch", C.c_int32), ("n_seq_max", C.c_int32), ("logit_softcap", C.c_float),
-                ("embed_scale", C.c_float), ("residual_mult", C.c_float)]
+                ("embed_scale", C.c_float), ("residual_mult", C.c_float), ("logit_scale", C.c_float)]
 
 
 class LayerParams(C.Structure):
@@ -36,7 +36,8 @@ class LayerParams(C.Structure):
                 ("glu_kind", C.c_int32), ("glu_limit", C.c_float), ("glu_alpha", C.c_float), ("router_score", C.c_int32), ("router_keep_scores", C.c_int32),
                 ("conv_taps", C.c_int32), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int32), ("dist_bias_max", C.c_int32), ("side_width", C.c_int32),
                 ("router_scale_input", C.c_int32), ("shared_ff", C.c_int32), ("loop_input", C.c_int32), ("dist_slope_exp", C.c_float), ("mix_heads", C.c_int32),
-                ("mix_dim", C.c_int32), ("left_scale", C.c_float), ("right_scale", C.c_float), ("token_side", C.c_int32)]
+                ("mix_dim", C.c_int32), ("left_scale", C.c_float), ("right_scale", C.c_float), ("token_side", C.c_int32),
+                ("attn_softcap", C.c_float), ("mix_kv_heads", C.c_int32), ("mix_vdim", C.c_int32), ("decay_rank", C.c_int32), ("gate_rank", C.c_int32), ("decay_tau", C.c_float)]
 
 
 _SIGS = {

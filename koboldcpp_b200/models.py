@@ -4,7 +4,7 @@ from __future__ import annotations
 import json
 from pathlib import Path
 
-from . import galirax, genesun, mafuzen, medodra, zevopel
+from . import galirax, genesun, mafuzen, medodra, tugezen, zevopel
 from .lib import B200Error
 
 ARCHITECTURES = {
@@ -13,6 +13,7 @@ ARCHITECTURES = {
     "Zevopel": zevopel.load,
     "Medodra": medodra.load,
     "Mafuzen": mafuzen.load,
+    "Tugezen": tugezen.load,
 }
 
 
