@@ -220,6 +220,8 @@ _OPS_SIGS = {
     "b200_op_sigmoid_mul": (C.c_int, [C.POINTER(Tensor), C.POINTER(Tensor), C.POINTER(Tensor), C.c_void_p]),
     "b200_op_latent_kv_store": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_int32, C.c_int32,
                                           C.c_int32, C.c_float, C.c_float, C.c_int32, C.c_void_p]),
+    "b200_op_latent_store": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_int32, C.c_int32,
+                                       C.c_int32, C.c_float, C.c_float, C.c_void_p, C.c_int64, C.c_void_p, C.c_int32, C.c_int32, C.c_void_p]),
     "b200_op_latent_attn": (C.c_int, [C.POINTER(LatentAttnArgs), C.c_void_p]),
     "b200_mlstm_state_floats": (C.c_int64, [C.c_int32, C.c_int32, C.c_int32]),
     "b200_op_mlstm_scan": (C.c_int, [C.POINTER(MlstmArgs), C.c_void_p]),
