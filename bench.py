@@ -937,13 +937,16 @@ def mafuzen_config(size: str) -> dict:
 
 def mafuzen_random_tensors(cfg: dict):
     W, V = cfg["width"], cfg["vocab"]
-    ES = cfg["token_side"]["dim"]
-    t = {"embed": (V, W), "final.norm": (W,), "final.norm.b": (W,), "side.embed": (V, ES * len(cfg["layers"]))}
+    ES = (cfg["token_side"] or {}).get("dim", 0)
+    t = {"embed": (V, W), "final.norm": (W,), "final.norm.b": (W,)}
+    if ES:
+        t["side.embed"] = (V, ES * len(cfg["layers"]))
     for i, L in enumerate(cfg["layers"]):
         p, mx = f"l{i}.", L["mixer"]
         for n in ("norm1", "norm1b", "norm2", "norm2b"):
             t.update({p + n: (W,), p + n + ".b": (W,)})
-        t.update({p + "side.gate": (ES, W), p + "side.proj": (W, ES), p + "side.norm": (W,)})
+        if ES:
+            t.update({p + "side.gate": (ES, W), p + "side.proj": (W, ES), p + "side.norm": (W,)})
         if L["type"] == "retention":
             H, D, Vd = mx["heads"], mx["dim"], mx["vdim"]
             t.update({p + "mix.q": (H * D, W), p + "mix.k": (H * D, W), p + "mix.v": (H * Vd, W), p + "mix.g": (H * Vd, W), p + "mix.o": (W, H * Vd)})
@@ -960,6 +963,10 @@ def mafuzen_random_tensors(cfg: dict):
             t.update({p + "mix.right." + x: (HD, W) for x in "rkvg"})
             t.update({p + "mix.right.w1": (MAFUZEN_RANK, W), p + "mix.right.w2": (HD, MAFUZEN_RANK), p + "mix.right.w0": (HD,), p + "mix.right.u": (mx["right"]["heads"], mx["right"]["dim"]),
                       p + "mix.right.norm": (HD,), p + "mix.right.o": (W, HD)})
+        if L["mlp"].get("kind") == "dense":
+            F = L["mlp"]["ff"]
+            t.update({p + "mlp.gate": (F, W), p + "mlp.up": (F, W), p + "mlp.down": (W, F)})
+            continue
         E, top, F, FS = L["mlp"]["router"]["experts"], L["mlp"]["router"]["top"], L["mlp"]["expert"]["ff"], L["mlp"]["shared"]["ff"]
         t.update({p + "mlp.shared.up": (FS, W), p + "mlp.shared.down": (W, FS), p + "mlp.table": (V, top)})
         for e in range(E):
@@ -983,7 +990,7 @@ def mafuzen_random_tensors(cfg: dict):
 def mafuzen_step_cost(cfg: dict, n_tokens: int, n_seq: int, ctx: int) -> dict:
     """Algorithmic bytes (bf16 weights once -- of the experts those a batch of this size can reach --, the visible f32 cache rows and the
     recurrent states of the batch) and FLOPs of one step."""
-    W, V, ES = cfg["width"], cfg["vocab"], cfg["token_side"]["dim"]
+    W, V, ES = cfg["width"], cfg["vocab"], (cfg["token_side"] or {}).get("dim", 0)
     wparams = active = W * V
     cache = state = attn_flop = 0
     for L in cfg["layers"]:
@@ -1007,6 +1014,10 @@ def mafuzen_step_cost(cfg: dict, n_tokens: int, n_seq: int, ctx: int) -> dict:
                 p += W * H * Vd + 5 * W * HR * DR + MAFUZEN_RANK * (W + HR * DR)  # the gate; r, k, v, g, o; the decay
                 state += n_seq * HR * DR * DR * 4 * 2
                 attn_flop += 4 * n_tokens * HR * DR * DR
+        if L["mlp"].get("kind") == "dense":
+            wparams += p + 3 * W * L["mlp"]["ff"] + 2 * W * ES
+            active += p + 3 * W * L["mlp"]["ff"] + 2 * W * ES
+            continue
         r, F, FS = L["mlp"]["router"], L["mlp"]["expert"]["ff"], L["mlp"]["shared"]["ff"]
         wparams += p + 2 * W * F * min(r["experts"], n_tokens * r["top"]) + 2 * W * FS + 2 * W * ES
         active += p + 2 * W * F * r["top"] + 2 * W * FS + 2 * W * ES
@@ -1023,6 +1034,103 @@ def mafuzen_beside_config(size: str) -> dict:
     lin = {"type": "lightning", "mixer": {"heads": h, "dim": d, "vdim": v, "decay": [1.0 - 2.0 ** (-5 - 3 * i / h) for i in range(h)]}, "mlp": mlp}
     win = {"type": "attention_2", "mixer": dict(att["mixer"], mask={"size": window, "keep_first": 4}), "mlp": mlp}
     return {"architecture": "Galirax", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": [(att, lin, win, att)[il % 4] for il in range(DESIGN_LAYERS)]}
+
+
+# ------------------------------------------------------------------------------------------------ --design tugezen
+# The same measurement for the Tugezen design (latent attention with a window, two layers of soft-capped attention beside the delta rule,
+# gated linear attention in turn; dense gated feed-forward), beside the closest existing model of the framework: Mafuzen with attention, two
+# layers of windowed attention beside time mixing, and retention in turn, at equal width, depth, heads and feed-forward size.
+TUGEZEN_GLA_RANK = 16
+
+
+def tugezen_config(size: str) -> dict:
+    import math
+    W, (h, g, d, v), _experts, window = GALIRAX_SIZES[size]
+    mlp = {"kind": "dense", "ff": 11 * W // 4}
+    sc = 1.0 / math.sqrt(d)
+    lat = {"type": "latent_attention", "mixer": {"heads": h, "dim": d, "vdim": v, "q_rank": 3 * W // 8, "kv_rank": 256 if W < 2048 else 512, "scale": sc, "mask": {"size": window}}, "mlp": mlp}
+    left = {"heads": h, "kv_heads": g, "dim": d, "vdim": v, "scale": sc, "softcap": 30.0,
+            "rot": {"base": 500000.0, "dims": d, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    par = {"type": "parallel", "mixer": {"left": left, "left_scale": 0.7, "right": {"heads": h, "kv_heads": h, "dim": 128, "vdim": 128, "conv": 4}, "right_scale": 0.8}, "mlp": mlp}
+    gla = {"type": "gla", "mixer": {"heads": h, "dim": d, "vdim": v, "tau": 16.0}, "mlp": mlp}
+    return {"architecture": "Tugezen", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-6}, "logit_scale": 0.5, "layers": [(lat, par, par, gla)[il % 4] for il in range(DESIGN_LAYERS)]}
+
+
+def tugezen_random_tensors(cfg: dict):
+    W, V = cfg["width"], cfg["vocab"]
+    t = {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+    for i, L in enumerate(cfg["layers"]):
+        p, mx, F = f"l{i}.", L["mixer"], L["mlp"]["ff"]
+        m = p + "mix."
+        t.update({p + "norm1": (W,), p + "norm2": (W,), p + "mlp.gate": (F, W), p + "mlp.up": (F, W), p + "mlp.down": (W, F)})
+        if L["type"] == "latent_attention":
+            H, D, Vd, QR, KR = (mx[k] for k in ("heads", "dim", "vdim", "q_rank", "kv_rank"))
+            t.update({m + "dq": (QR, W), m + "dq.norm": (QR,), m + "uq": (H * D, QR), m + "dkv": (KR, W), m + "dkv.norm": (KR,), m + "uk": (H * D, KR), m + "uv": (H * Vd, KR), m + "g": (H, W),
+                      m + "o": (W, H * Vd)})
+        elif L["type"] == "gla":
+            H, D, Vd = mx["heads"], mx["dim"], mx["vdim"]
+            t.update({m + "q": (H * D, W), m + "k": (H * D, W), m + "v": (H * Vd, W), m + "g": (H * Vd, W), m + "o": (W, H * Vd), m + "norm": (Vd,), m + "a1": (TUGEZEN_GLA_RANK, W),
+                      m + "a2": (H * D, TUGEZEN_GLA_RANK), m + "a2.b": (H * D,)})
+        else:
+            a, r = mx["left"], mx["right"]
+            H, G, D, Vd = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            t.update({m + "left.q": (H * D, W), m + "left.k": (G * D, W), m + "left.v": (G * Vd, W), m + "left.o": (W, H * Vd)})
+            H, G, D, Vd, rank = r["heads"], r["kv_heads"], r["dim"], r["vdim"], r["vdim"]
+            m += "right."
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * Vd)):
+                t.update({m + n: (rows, W), m + n + ".conv": (rows, r["conv"])})
+            t.update({m + "b": (H, W), m + "A_log": (H,), m + "dt_bias": (H * D,), m + "norm": (Vd,), m + "a1": (rank, W), m + "a2": (H * D, rank), m + "g1": (rank, W), m + "g2": (H * Vd, rank),
+                      m + "o": (W, H * Vd)})
+    out = random_tensors(t)
+    for name, shape in t.items():
+        if name.endswith(".dt_bias"):  # decays between 0.5 and 0.999
+            out[name] = ("F32", shape, np.linspace(-7.0, 0.0, shape[0], dtype=np.float32).view(np.uint8))
+    return out
+
+
+def tugezen_step_cost(cfg: dict, n_tokens: int, n_seq: int, ctx: int) -> dict:
+    """Algorithmic bytes (bf16 weights once, the visible f32 cache rows and the recurrent states of the batch) and FLOPs of one step."""
+    W, V = cfg["width"], cfg["vocab"]
+    params = W * V
+    cache = state = attn_flop = 0
+    full = ctx if n_tokens == n_seq else ctx // 2
+    for L in cfg["layers"]:
+        mx = L["mixer"]
+        if L["type"] == "latent_attention":
+            H, D, Vd, QR, KR = (mx[k] for k in ("heads", "dim", "vdim", "q_rank", "kv_rank"))
+            vis = min(ctx, mx["mask"]["size"])
+            params += W * (QR + KR + H) + H * D * QR + H * (D + Vd) * KR + W * H * Vd
+            cache += n_seq * vis * KR * 4
+            attn_flop += 2 * n_tokens * H * min(vis, full) * 2 * KR
+        elif L["type"] == "gla":
+            H, D, Vd = mx["heads"], mx["dim"], mx["vdim"]
+            params += W * (2 * H * D + 2 * H * Vd) + W * H * Vd + TUGEZEN_GLA_RANK * (W + H * D)
+            state += n_seq * H * D * Vd * 4 * 2
+            attn_flop += 4 * n_tokens * H * D * Vd
+        else:
+            a, r = mx["left"], mx["right"]
+            H, G, D, Vd = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            params += W * (H * D + G * D + G * Vd + H * Vd)
+            cache += n_seq * ctx * G * (D + Vd) * 4
+            attn_flop += 2 * n_tokens * H * full * (D + Vd)
+            H, G, D, Vd = r["heads"], r["kv_heads"], r["dim"], r["vdim"]
+            params += W * (2 * G * D + 2 * H * Vd + H) + Vd * (2 * W + H * D + H * Vd)
+            state += n_seq * H * D * Vd * 4 * 2
+            attn_flop += 6 * n_tokens * H * D * Vd
+        params += 3 * W * L["mlp"]["ff"]
+    return {"weight_bytes": 2 * params, "cache_bytes": cache, "state_bytes": state, "flop": 2 * params * n_tokens + attn_flop}
+
+
+def tugezen_beside_config(size: str) -> dict:
+    """Mafuzen at equal width, depth, heads and feed-forward: attention, two parallel layers and retention in turn, no token input."""
+    import math
+    W, (h, g, d, v), _experts, window = GALIRAX_SIZES[size]
+    mlp = {"kind": "dense", "ff": 11 * W // 4}
+    att = {"heads": h, "kv_heads": g, "dim": d, "vdim": v, "scale": 1.0 / math.sqrt(d)}
+    a = {"type": "attention", "mixer": att, "mlp": mlp}
+    par = {"type": "parallel", "mixer": {"left": dict(att, mask={"size": window, "keep_first": 4}), "left_scale": 0.7, "right": {"heads": W // 64, "dim": 64}, "right_scale": 0.8}, "mlp": mlp}
+    ret = {"type": "retention", "mixer": {"heads": h, "dim": d, "vdim": v, "rot": {"base": 10000.0, "dims": d}, "decay": [1.0 - 2.0 ** (-5 - 3 * i / h) for i in range(h)]}, "mlp": mlp}
+    return {"architecture": "Mafuzen", "width": W, "vocab": DESIGN_VOCAB, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "token_side": None, "layers": [(a, par, par, ret)[il % 4] for il in range(DESIGN_LAYERS)]}
 
 
 def galirax_llama_shape(size: str):
@@ -1062,8 +1170,11 @@ def random_tensors(shapes: dict, seed: int = 1):
 
 
 def design_table():
-    from koboldcpp_b200 import galirax, genesun, mafuzen, medodra, zevopel
+    from koboldcpp_b200 import galirax, genesun, mafuzen, medodra, tugezen, zevopel
     return {
+        "tugezen": {"sizes": GALIRAX_SIZES, "config": tugezen_config, "tensors": tugezen_random_tensors, "cost": tugezen_step_cost, "build": tugezen.build,
+                    "beside_design": {"name": "mafuzen", "config": tugezen_beside_config, "tensors": mafuzen_random_tensors, "cost": mafuzen_step_cost, "build": mafuzen.build},
+                    "beside": "Mafuzen (attention, two layers of windowed attention beside time mixing, retention in turn, dense gated feed-forward), equal width / depth / heads / ff, bf16"},
         "mafuzen": {"sizes": GALIRAX_SIZES, "config": mafuzen_config, "tensors": mafuzen_random_tensors, "cost": mafuzen_step_cost, "build": mafuzen.build,
                     "beside_design": {"name": "galirax", "config": mafuzen_beside_config, "tensors": lambda cfg: random_tensors(galirax_tensor_shapes(cfg)),
                                       "cost": galirax_step_cost, "build": galirax.build},
@@ -1203,7 +1314,7 @@ def main() -> int:
     ap.add_argument("--cpu-budget", type=float, default=18.0)
     ap.add_argument("--no-tp70", action="store_true", default=bool(os.environ.get("B200_BENCH_NO_TP70")),
                     help="skip the auxiliary 70B tensor-parallel leg (BASELINE.json configs[4])")
-    ap.add_argument("--design", default="", choices=["", "genesun", "galirax", "zevopel", "medodra", "mafuzen"],
+    ap.add_argument("--design", default="", choices=["", "genesun", "galirax", "zevopel", "medodra", "mafuzen", "tugezen"],
                     help="instead of the default workload: prefill / decode of this design at real layer shapes beside the closest existing model at equal size")
     ap.add_argument("--design-sizes", default="", help="comma-separated subset of the sizes of the design (genesun: " + ",".join(DESIGN_SIZES) + "; the others: " + ",".join(GALIRAX_SIZES) + ")")
     args = ap.parse_args()
