@@ -567,6 +567,7 @@ __device__ __forceinline__ float la_channel_decay(float z, float inv_tau) { retu
 template <int DPL, bool CHAN>
 __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b200_linear_attn_args a) {
     constexpr int LA_CHUNK = la_chunk<DPL, CHAN>();
+    __shared__ float sb[CHAN ? 32 * DPL : 1];  // z_bias of the head (not added where z is read: the test of the pointer would make those loads wait for one another)
     extern __shared__ float sm_[];  // q [LA_CHUNK][32 DPL], k [LA_CHUNK][32 DPL], v [LA_CHUNK][LA_COLS], with CHAN decays [LA_CHUNK][32 DPL]
     const int h = blockIdx.y, s = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
@@ -597,7 +598,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
             const int64_t tok = first + t0 + tt;
             pq[j] = ok ? a.q[tok * a.q_stride + (int64_t)h * D + d] : 0.f;
             pk[j] = ok ? a.k[tok * a.k_stride + (int64_t)h * D + d] : 0.f;
-            if (CHAN) pz[CHAN ? j : 0] = ok ? a.z[tok * a.z_stride + (int64_t)h * D + d] + (a.z_bias ? a.z_bias[h * D + d] : 0.f) : 0.f;
+            if (CHAN) pz[CHAN ? j : 0] = ok ? a.z[tok * a.z_stride + (int64_t)h * D + d] : 0.f;
         }
 #pragma unroll
         for (int j = 0; j < NVV; j++) {
@@ -606,6 +607,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
         }
     };
     fetch(0);
+    if (CHAN) for (int d = tid; d < DP; d += LA_WARPS * 32) sb[d] = a.z_bias && d < D ? a.z_bias[(int64_t)h * D + d] : 0.f;
     for (int t0 = 0; t0 < count; t0 += LA_CHUNK) {
         const int nt = min(LA_CHUNK, count - t0);
         __syncthreads();  // the previous chunk has been read
@@ -615,7 +617,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) linear_attn_scan_kernel(const b
         for (int j = 0; j < NVV; j++) sv[tid + j * LA_WARPS * 32] = la_act(pv[j], a.act);
         if (CHAN) {
 #pragma unroll
-            for (int j = 0; j < NQ; j++) sw[tid + j * LA_WARPS * 32] = la_channel_decay(pz[CHAN ? j : 0], inv_tau);
+            for (int j = 0; j < NQ; j++) sw[tid + j * LA_WARPS * 32] = la_channel_decay(pz[CHAN ? j : 0] + sb[CHAN ? (tid + j * LA_WARPS * 32) % DP : 0], inv_tau);
         }
         __syncthreads();
         if (a.n_dims > 0) {  // rotation of entry i with entry i + n_dims / 2 where the rows wait (the scale on k commutes with it)

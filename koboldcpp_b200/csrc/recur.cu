@@ -77,6 +77,7 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
     constexpr int DP = 32 * DQ, DR_CHUNK = CHAN && DQ > 4 ? 8 : 16, DR_TPW = DR_CHUNK / DR_WARPS;  // (three staged rows of 256 values: half the tokens fit)
     __shared__ __align__(16) float sq[DR_CHUNK][DP], sk[DR_CHUNK][DP];
     __shared__ __align__(16) float sgc[CHAN ? DR_CHUNK : 1][CHAN ? DP : 4];
+    __shared__ float sbias[CHAN ? DP : 1];  // (not added where a.a is read: the test of the pointer would make those loads wait for one another)
     __shared__ float sv[DR_CHUNK][DR_COLS], sqk[DR_CHUNK], sg[DR_CHUNK], sbeta[DR_CHUNK];
     const int h = blockIdx.y, s = blockIdx.z, kvh = h / (a.heads / a.kv_heads);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
@@ -109,7 +110,7 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
             const int64_t tok = first + t0 + tt;
             pq[j] = ok ? a.q[tok * a.q_stride + (int64_t)kvh * D + d] : 0.f;
             pk[j] = ok ? a.k[tok * a.k_stride + (int64_t)kvh * D + d] : 0.f;
-            if (CHAN) pg[CHAN ? j : 0] = ok ? a.a[tok * a.a_stride + (int64_t)h * D + d] + (a.dt_bias ? a.dt_bias[(int64_t)h * D + d] : 0.f) : 0.f;
+            if (CHAN) pg[CHAN ? j : 0] = ok ? a.a[tok * a.a_stride + (int64_t)h * D + d] : 0.f;
         }
 #pragma unroll
         for (int j = 0; j < NVV; j++) {
@@ -122,6 +123,7 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
         }
     };
     fetch(0);
+    if (CHAN) for (int d = tid; d < DP; d += DR_WARPS * 32) sbias[d] = a.dt_bias && d < D ? a.dt_bias[(int64_t)h * D + d] : 0.f;
     for (int t0 = 0; t0 < count; t0 += DR_CHUNK) {
         const int nt = min(DR_CHUNK, count - t0);
         __syncthreads();  // the previous chunk has been read
@@ -131,7 +133,7 @@ __global__ void __launch_bounds__(DR_WARPS * 32) delta_rule_scan_kernel(const b2
         for (int j = 0; j < NVV; j++) (&sv[0][0])[tid + j * DR_WARPS * 32] = pv[j];
         if (CHAN) {
 #pragma unroll
-            for (int j = 0; j < NQ; j++) (&sgc[0][0])[tid + j * DR_WARPS * 32] = expf(-decay_rate * softplus_f(pg[CHAN ? j : 0]));
+            for (int j = 0; j < NQ; j++) (&sgc[0][0])[tid + j * DR_WARPS * 32] = expf(-decay_rate * softplus_f(pg[CHAN ? j : 0] + sbias[CHAN ? (tid + j * DR_WARPS * 32) % DP : 0]));
         }
         if (tid < DR_CHUNK) {
             if (!CHAN) sg[tid] = expf(-decay_rate * softplus_f(pa + dtb));
