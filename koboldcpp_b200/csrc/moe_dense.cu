@@ -201,6 +201,22 @@ __global__ void glu_strided_kernel(TD a, TD b, TD sc, bool has_scale, TD dst, in
     *(float *)(dst.data + i0 * dst.nb[0] + i1 * dst.nb[1] + i2 * dst.nb[2] + i3 * dst.nb[3]) = glu_value<KIND>(x, u, limit, alpha);
 }
 
+// contiguous values in every row and 16-byte aligned rows: 4 values a thread, the row's place from the grid instead of divisions
+template <int KIND>
+__global__ void __launch_bounds__(256) glu_rows_kernel(TD a, TD b, TD sc, bool has_scale, TD dst, int n4, float limit, float alpha) {
+    const int i = blockIdx.x * 256 + threadIdx.x;
+    const int64_t i1 = blockIdx.y, i2 = blockIdx.z;
+    if (i >= n4) return;
+    float4 x = reinterpret_cast<const float4 *>(a.data + i1 * a.nb[1] + i2 * a.nb[2])[i], u = reinterpret_cast<const float4 *>(b.data + i1 * b.nb[1] + i2 * b.nb[2])[i];
+    if (has_scale) {
+        const float f = *(const float *)(sc.data + i1 * sc.nb[0] + i2 * sc.nb[1]);
+        x.x *= f; x.y *= f; x.z *= f; x.w *= f;
+        u.x *= f; u.y *= f; u.z *= f; u.w *= f;
+    }
+    reinterpret_cast<float4 *>(dst.data + i1 * dst.nb[1] + i2 * dst.nb[2])[i] =
+        make_float4(glu_value<KIND>(x.x, u.x, limit, alpha), glu_value<KIND>(x.y, u.y, limit, alpha), glu_value<KIND>(x.z, u.z, limit, alpha), glu_value<KIND>(x.w, u.w, limit, alpha));
+}
+
 __global__ void moe_combine_kernel(const float *__restrict__ y, int64_t y_s_slot, int64_t y_s_tok, const float *__restrict__ w, int64_t w_s_tok,
                                    const float *__restrict__ add0, int64_t add0_stride, const float *__restrict__ add1, int64_t add1_stride, float *__restrict__ dst,
                                    int64_t dst_stride, int64_t n, int n_used, int64_t total) {
@@ -378,9 +394,18 @@ extern "C" int b200_op_glu_scaled(int kind, const b200_tensor *a, const b200_ten
     const int64_t n = nelements(dst);
     if (n == 0) return B200_OK;
     const cudaStream_t st = (cudaStream_t)stream;
-    if (kind == B200_GLU_GELU_TANH) glu_strided_kernel<B200_GLU_GELU_TANH><<<grid1d(n, 256), 256, 0, st>>>(td(a), td(b), tsc, scale != nullptr, td(dst), n, limit, alpha);
-    else if (kind == B200_GLU_SWISH_CLAMPED) glu_strided_kernel<B200_GLU_SWISH_CLAMPED><<<grid1d(n, 256), 256, 0, st>>>(td(a), td(b), tsc, scale != nullptr, td(dst), n, limit, alpha);
-    else glu_strided_kernel<B200_GLU_SILU><<<grid1d(n, 256), 256, 0, st>>>(td(a), td(b), tsc, scale != nullptr, td(dst), n, limit, alpha);
+    auto rows16 = [](const b200_tensor *t) { return t->nb[0] == 4 && (((uintptr_t)t->data | t->nb[1] | t->nb[2]) & 15) == 0; };
+    const bool vec = dst->ne[0] % 4 == 0 && dst->ne[0] <= 0x7fffffff && dst->ne[1] <= 65535 && dst->ne[2] <= 65535 && dst->ne[3] == 1 && rows16(a) && rows16(b) && rows16(dst);
+    const dim3 grid((unsigned)((dst->ne[0] / 4 + 255) / 256), (unsigned)dst->ne[1], (unsigned)dst->ne[2]);
+#define B200_GLU(K)                                                                                                                                           \
+    do {                                                                                                                                                      \
+        if (vec) glu_rows_kernel<K><<<grid, 256, 0, st>>>(td(a), td(b), tsc, scale != nullptr, td(dst), (int)(dst->ne[0] / 4), limit, alpha);                 \
+        else glu_strided_kernel<K><<<grid1d(n, 256), 256, 0, st>>>(td(a), td(b), tsc, scale != nullptr, td(dst), n, limit, alpha);                            \
+    } while (0)
+    if (kind == B200_GLU_GELU_TANH) B200_GLU(B200_GLU_GELU_TANH);
+    else if (kind == B200_GLU_SWISH_CLAMPED) B200_GLU(B200_GLU_SWISH_CLAMPED);
+    else B200_GLU(B200_GLU_SILU);
+#undef B200_GLU
     B200_CUDA_TRY(cudaGetLastError());
     return B200_OK;
 }

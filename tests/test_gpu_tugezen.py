@@ -63,13 +63,17 @@ def test_head_norm_with_one_weight_for_all_heads_and_a_gate(V, Hh, T, gate):
         assert rel(got[:, h], want[:, h]) < 3e-6
 
 
-def test_gated_activation_with_the_tanh_form_of_gelu():
-    a, b = np.linspace(-9, 9, 3 * 37).reshape(3, 37), np.random.default_rng(0).standard_normal((3, 37))
+@pytest.mark.parametrize("F,T,kind", [(37, 3, 1), (64, 3, 1), (1028, 2, 1), (2052, 3, 0), (36, 2, 2)])
+def test_gated_activation_rows_of_four_and_others(F, T, kind):
+    """The tanh form of gelu (1), and the other kinds through the same forms, over the halves of one product."""
+    a, b = np.linspace(-9, 9, T * F).reshape(T, F), np.random.default_rng(0).standard_normal((T, F)) * 3
     gu, out = dev(np.concatenate([a, b], 1)), H.DeviceBuffer(4 * a.size + 256)
-    ta, tb, to = Tensor.contiguous(gu.ptr, F32, (37, 3)), Tensor.contiguous(gu.ptr + 4 * 37, F32, (37, 3)), Tensor.contiguous(out.ptr, F32, (37, 3))
-    ta.nb[1] = tb.nb[1] = 4 * 74
-    check(lib().b200_op_glu_strided(1, C.byref(ta), C.byref(tb), C.byref(to), 0.0, 0.0, None))
-    assert rel(out.to_numpy(np.float32, (3, 37)), R.gelu_tanh(a) * b) < 2e-6
+    ta, tb, to = Tensor.contiguous(gu.ptr, F32, (F, T)), Tensor.contiguous(gu.ptr + 4 * F, F32, (F, T)), Tensor.contiguous(out.ptr, F32, (F, T))
+    ta.nb[1] = tb.nb[1] = 8 * F
+    check(lib().b200_op_glu_strided(kind, C.byref(ta), C.byref(tb), C.byref(to), 5.0, 1.5, None))
+    g, u = np.minimum(a, 5.0), np.clip(b, -5.0, 5.0)
+    want = (R.silu(a) * b, R.gelu_tanh(a) * b, g * R.sigmoid(1.5 * g) * (u + 1.0))[kind]
+    assert rel(out.to_numpy(np.float32, (T, F)), want) < 2e-6
 
 
 # ------------------------------------------------------------------------------------------------ recurrences
