@@ -38,7 +38,17 @@ __global__ void __launch_bounds__(128) short_conv_kernel(const b200_short_conv_a
 #pragma unroll
         for (int j = 0; j < KMAX; j++) wp[j] = j >= KMAX - taps ? w[j - (KMAX - taps)] : 0.f;
 #pragma unroll
-        for (int i = 0; i < SC_TOK + KMAX - 1; i++) win[i] = i - (KMAX - 1) < nt ? input(t0 + i - (KMAX - 1)) : 0.f;  // win[i] = input t0 + i - (KMAX - 1)
+        for (int i = 0; i < SC_TOK + KMAX - 1; i++) win[i] = 0.f;  // win[i] = input t0 + i - (KMAX - 1)
+        if (t0 > 0) {  // every input is a value of x (KMAX - 1 <= SC_TOK): no test between the loads but the end of the portion
+            const float *xp = a.x + (int64_t)(first + t0 - (KMAX - 1)) * a.x_stride + c;
+#pragma unroll
+            for (int i = 0; i < SC_TOK + KMAX - 1; i++) if (i - (KMAX - 1) < nt) win[i] = xp[(int64_t)i * a.x_stride];
+#pragma unroll
+            for (int i = 0; i < SC_TOK + KMAX - 1; i++) win[i] += bias;  // (beyond the portion's end nobody reads it)
+        } else {
+#pragma unroll
+            for (int i = 0; i < SC_TOK + KMAX - 1; i++) if (i - (KMAX - 1) < nt) win[i] = input(t0 + i - (KMAX - 1));
+        }
 #pragma unroll
         for (int t = 0; t < SC_TOK; t++) {
             float y = 0.f;
